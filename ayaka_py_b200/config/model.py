@@ -468,3 +468,108 @@ class TesozenConfig(ModelConfig):
         return {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width,
                 "layers": [json.loads(json.dumps(layer)) for layer in self.layers], "norm": dict(self.norm),
                 "embedding": dict(self.embedding)}
+
+
+_MURUTAR_MIXERS = {"attention": ("heads", "kv_heads", "dim", "vdim"), "lightning": ("heads", "dim", "vdim")}
+
+
+@dataclass(frozen=True)
+class MurutarConfig(ModelConfig):
+    """Murutar: ``layers`` lists the layers in order, each {"type": "attention" | "lightning", "mixer": its sizes
+    and constants, "mlp": {"kind": "dense", "ff": n, "limit": c}, {"kind": "moe", "router": {experts, top, groups:
+    {count, keep}}, "expert": {ff}} or null}.  ``attention``: heads, kv_heads, dim, vdim, scale, rot {dims, base},
+    mask.size (the window) and v_mix; ``lightning``: heads, dim, vdim and a decay per head.  ``norm.eps``,
+    ``embedding.scale``, ``token_side.dim`` (columns of the side table per layer) and ``logit_softcap`` are the
+    model-wide constants.  The document names the design under ``architecture``.  The model has no position
+    limit of its own."""
+
+    ARCHITECTURE: ClassVar[str] = "Murutar"
+
+    vocab: int = 0
+    width: int = 0
+    layers: tuple = ()
+    norm: Mapping[str, Any] = dataclasses.field(default_factory=lambda: {"eps": 1e-6})
+    embedding: Mapping[str, Any] = dataclasses.field(default_factory=lambda: {"scale": 1.0})
+    token_side: Mapping[str, Any] = dataclasses.field(default_factory=dict)
+    logit_softcap: float = 30.0
+
+    def __post_init__(self) -> None:
+        _require_int(self.vocab, "vocab")
+        _require_int(self.width, "width")
+        if not isinstance(self.layers, (list, tuple)) or not self.layers:
+            raise ConfigError("layers must be a non-empty list")
+        object.__setattr__(self, "layers", tuple(self.layers))
+        _require_number(self.norm.get("eps") if isinstance(self.norm, Mapping) else None, "norm.eps", positive=True)
+        _require_number(self.embedding.get("scale") if isinstance(self.embedding, Mapping) else None, "embedding.scale")
+        _require_int(self.token_side.get("dim") if isinstance(self.token_side, Mapping) else None, "token_side.dim")
+        _require_number(self.logit_softcap, "logit_softcap", positive=True)
+        value_widths = set()
+        for i, layer in enumerate(self.layers):
+            kind = layer.get("type") if isinstance(layer, Mapping) else None
+            if kind not in _MURUTAR_MIXERS:
+                raise ConfigError(f"layers[{i}].type must be one of {sorted(_MURUTAR_MIXERS)}, got {kind!r}")
+            mixer = layer.get("mixer")
+            if not isinstance(mixer, Mapping):
+                raise ConfigError(f"layers[{i}].mixer must give the mixer's sizes")
+            for key in _MURUTAR_MIXERS[kind]:
+                _require_int(mixer.get(key), f"layers[{i}].mixer.{key}")
+            if kind == "attention":
+                if mixer["heads"] % mixer["kv_heads"]:
+                    raise ConfigError(f"layers[{i}].mixer: {mixer['heads']} heads cannot share {mixer['kv_heads']} key/value heads")
+                _require_number(mixer.get("scale"), f"layers[{i}].mixer.scale")
+                rot = mixer.get("rot")
+                if not isinstance(rot, Mapping):
+                    raise ConfigError(f"layers[{i}].mixer.rot must give the rotation's constants")
+                dims = _require_int(rot.get("dims"), f"layers[{i}].mixer.rot.dims")
+                _require_number(rot.get("base"), f"layers[{i}].mixer.rot.base", positive=True)
+                if dims % 2 or dims > mixer["dim"]:
+                    raise ConfigError(f"layers[{i}].mixer.rot.dims must be even and at most dim")
+                mask = mixer.get("mask")
+                if mask is not None:
+                    if not isinstance(mask, Mapping):
+                        raise ConfigError(f"layers[{i}].mixer.mask must give the window's size")
+                    _require_int(mask.get("size"), f"layers[{i}].mixer.mask.size")
+                mixes = mixer.get("v_mix", False)
+                if not isinstance(mixes, bool):
+                    raise ConfigError(f"layers[{i}].mixer.v_mix must be true or false")
+                if mixes:
+                    value_widths.add((mixer["kv_heads"], mixer["vdim"]))
+            else:
+                decay = mixer.get("decay")
+                if not isinstance(decay, (list, tuple)) or len(decay) != mixer["heads"]:
+                    raise ConfigError(f"layers[{i}].mixer.decay must give one number per head")
+                for h, value in enumerate(decay):
+                    if not 0.0 <= _require_number(value, f"layers[{i}].mixer.decay[{h}]") <= 1.0:
+                        raise ConfigError(f"layers[{i}].mixer.decay[{h}] must lie between 0 and 1, got {value}")
+            mlp = layer.get("mlp")
+            if mlp is None:
+                continue
+            if not isinstance(mlp, Mapping) or mlp.get("kind") not in ("dense", "moe"):
+                raise ConfigError(f"layers[{i}].mlp.kind must be 'dense' or 'moe' (or mlp null), got {mlp!r}")
+            if mlp["kind"] == "dense":
+                _require_int(mlp.get("ff"), f"layers[{i}].mlp.ff")
+                _require_number(mlp.get("limit"), f"layers[{i}].mlp.limit", positive=True)
+                continue
+            router, expert = mlp.get("router"), mlp.get("expert")
+            if not isinstance(router, Mapping) or not isinstance(expert, Mapping):
+                raise ConfigError(f"layers[{i}].mlp must give router and expert")
+            experts = _require_int(router.get("experts"), f"layers[{i}].mlp.router.experts")
+            top = _require_int(router.get("top"), f"layers[{i}].mlp.router.top")
+            _require_int(expert.get("ff"), f"layers[{i}].mlp.expert.ff")
+            groups = router.get("groups")
+            count = keep = 1
+            if groups is not None:
+                if not isinstance(groups, Mapping):
+                    raise ConfigError(f"layers[{i}].mlp.router.groups must give count and keep")
+                count = _require_int(groups.get("count"), f"layers[{i}].mlp.router.groups.count")
+                keep = _require_int(groups.get("keep"), f"layers[{i}].mlp.router.groups.keep")
+            if experts % count or keep > count or keep * (experts // count) < top or top > experts:
+                raise ConfigError(f"layers[{i}].mlp.router: {experts} experts in {count} groups of which {keep} are kept "
+                                  f"cannot give {top} choices")
+        if len(value_widths) > 1:
+            raise ConfigError(f"layers that mix values must have equal kv_heads and vdim, got {sorted(value_widths)}")
+
+    def to_dict(self) -> dict[str, Any]:
+        return {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width,
+                "layers": [json.loads(json.dumps(layer)) for layer in self.layers], "norm": dict(self.norm),
+                "embedding": dict(self.embedding), "token_side": dict(self.token_side), "logit_softcap": self.logit_softcap}

@@ -15,6 +15,7 @@ struct GroupedArgs {
   const int* req_q_start;
   const int* req_pos0;
   const float* slopes;       // [QH] or null
+  const float* sinks;        // [QH] or null: the score of one more key without a value, in every row's denominator
   const float* gate;         // float32 rows whose first QH * DV numbers gate the output, or null
   long long gate_stride;
   int table_stride, num_req, total_rows;
@@ -22,12 +23,18 @@ struct GroupedArgs {
   int window, keep_first;    // window <= 0: every earlier key
   int chunk;                 // > 0: only keys of the query's own run of ``chunk`` positions (runs counted from position 0)
   int parts, part_keys;      // part_keys 0: the context is not cut
+  int parts_from_window;     // the parts are counted from the one that holds the window's first key, not from key 0
   float scale;
 };
 
 // Does the query at position i see the key at position j?
 __host__ __device__ __forceinline__ bool grouped_visible(int i, int j, int window, int keep_first, int chunk = 0) {
   return j <= i && (window <= 0 || i - j < window || j < keep_first) && (chunk <= 0 || j >= i / chunk * chunk);
+}
+
+// The part that a row's first part (grid index 0) is, when parts are counted from its window's first key.
+__host__ __device__ __forceinline__ int grouped_base_part(int pos, int window, int part_keys) {
+  return pos >= window ? (pos - window + 1) / part_keys : 0;
 }
 
 // Tiles of ``step`` keys from k_first on that hold a key some row of the block may see: those below

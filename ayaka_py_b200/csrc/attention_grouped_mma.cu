@@ -73,7 +73,8 @@ grouped_attention_mma_kernel(GroupedArgs a, int page_shift, int tq, int DKP, int
   const int pos0 = a.req_pos0[req] + q0;
   const int last_pos = pos0 + tokens - 1;
   const int part = blockIdx.z;
-  const int k_first = a.part_keys > 0 ? part * a.part_keys : 0;
+  const int base_part = a.parts_from_window ? grouped_base_part(pos0, a.window, a.part_keys) : 0;
+  const int k_first = a.part_keys > 0 ? (base_part + part) * a.part_keys : 0;
   const int k_last = a.part_keys > 0 ? min(last_pos, k_first + a.part_keys - 1) : last_pos;
   if (k_first > last_pos) return;                   // the merge does not read parts beyond the context
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
@@ -154,6 +155,15 @@ grouped_attention_mma_kernel(GroupedArgs a, int page_shift, int tq, int DKP, int
 #pragma unroll
     for (int c = 0; c < 4; ++c) o[nt][c] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};     // l: this thread's share of the row's denominator
+  if (a.sinks && part == 0) {                          // the sink counts once per row: in the first part, one of the row's four threads
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int m = warp * 16 + gid + half * 8;
+      if (m >= rows) continue;
+      m_run[half] = a.sinks[g * hpg + m % hpg] * LOG2E;
+      l_run[half] = tig == 0 ? 1.f : 0.f;
+    }
+  }
   const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(Qs + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDK + (lane >> 4) * 8);
   const int ksteps = DKP / 16;
 

@@ -87,6 +87,7 @@ __device__ __forceinline__ float apply_activation_tc(float x, int act) {
     const float r = fmaxf(x, 0.0f);
     return r * r;
   }
+  if (ACT == AYK_ACT_SILU) return __fdividef(x, 1.0f + fast_exp2(-1.4426950408889634f * x));
   return apply_activation(x, act);
 }
 

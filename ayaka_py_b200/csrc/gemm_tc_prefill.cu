@@ -105,11 +105,12 @@ __device__ __forceinline__ long long cache_place(const PrefillArgs& a, int row) 
 // uses are compiled on their own (MODE): 0 = bfloat16 out, no activation, no residual; 1 = float32
 // out with residual; 2 = bfloat16 out with tanh-GELU; 3 = anything, decided at run time; 4 = as 0, and
 // the key and value columns go into the paged cache as well (`place`: where this row's do, or -1); 5 = bfloat16
-// out with the squared ReLU.
+// out with the squared ReLU; 6 = bfloat16 out with SiLU.
 template <int W, int MODE>
 __device__ __forceinline__ void epilogue_chunk(const PrefillArgs& a, uint32_t taddr, int row, int n, bool row_ok,
                                                long long place) {
-  constexpr int ACT = MODE == 2 ? AYK_ACT_GELU_TANH : (MODE == 5 ? AYK_ACT_RELU2 : (MODE == 3 ? -1 : AYK_ACT_NONE));
+  constexpr int ACT = MODE == 2 ? AYK_ACT_GELU_TANH
+                    : (MODE == 5 ? AYK_ACT_RELU2 : (MODE == 6 ? AYK_ACT_SILU : (MODE == 3 ? -1 : AYK_ACT_NONE)));
   uint32_t r[W];
   if (W == 32) tmem_ld32(taddr, r); else tmem_ld16(taddr, r);
   const size_t idx = (size_t)row * a.N + n;
@@ -202,6 +203,7 @@ __device__ __forceinline__ void epilogue_row_any(const PrefillArgs& a, uint32_t 
   else if (a.mode == 2) epilogue_row<2>(a, taddr, row, n, cols, row_ok, place);
   else if (a.mode == 4) epilogue_row<4>(a, taddr, row, n, cols, row_ok, place);
   else if (a.mode == 5) epilogue_row<5>(a, taddr, row, n, cols, row_ok, place);
+  else if (a.mode == 6) epilogue_row<6>(a, taddr, row, n, cols, row_ok, place);
   else epilogue_row<3>(a, taddr, row, n, cols, row_ok, place);
 }
 
@@ -983,6 +985,7 @@ int epilogue_mode(int act, bool with_residual, bool out_bf16) {
   if (act == AYK_ACT_NONE && !out_bf16) return 1;
   if (act == AYK_ACT_GELU_TANH && !with_residual && out_bf16) return 2;
   if (act == AYK_ACT_RELU2 && !with_residual && out_bf16) return 5;
+  if (act == AYK_ACT_SILU && !with_residual && out_bf16) return 6;
   return 3;
 }
 
@@ -1279,9 +1282,9 @@ int prefill_product(void* C, const void* X, const void* W, const float* bias, co
 
 // Grouped product: X [M, K] in tiles of 128 rows, each tile's rows multiplied by the matrix that starts at
 // weight row w_rows[tile] of W [w_total_rows, K] (matrices of N rows one after the other); C [M, N], bfloat16
-// or float32, no bias, activation or residual.  M is a multiple of 128.  Whole tiles only (no split along K).
+// or float32, with an activation but no bias or residual.  M is a multiple of 128.  Whole tiles only (no split along K).
 AYK_EXPORT int ayk_gemm_tc_prefill_grouped(void* C, const void* X, const void* W, const int* w_rows, int M, int N, int K,
-                                           int w_total_rows, int out_dtype, int sms, cudaStream_t stream) {
+                                           int w_total_rows, int act, int out_dtype, int sms, cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   AYK_REQUIRE(M % BM == 0 && K % 8 == 0 && w_rows != nullptr, "ayk_gemm_tc_prefill_grouped: rows in whole tiles of %d, K a multiple of 8", BM);
   AYK_REQUIRE((uintptr_t)X % 16 == 0 && (uintptr_t)W % 16 == 0 && (uintptr_t)C % 16 == 0, "ayk_gemm_tc_prefill_grouped: operands must be 16-byte aligned");
@@ -1307,10 +1310,10 @@ AYK_EXPORT int ayk_gemm_tc_prefill_grouped(void* C, const void* X, const void* W
   }
   PrefillArgs args{};
   args.C = C; args.error = g_error_dev;
-  args.M = M; args.N = N; args.K = K; args.act = AYK_ACT_NONE; args.out_bf16 = out_dtype == AYK_DTYPE_BF16;
+  args.M = M; args.N = N; args.K = K; args.act = act; args.out_bf16 = out_dtype == AYK_DTYPE_BF16;
   args.BN = BN;
   args.vec_ok = N % 8 == 0;
-  args.mode = epilogue_mode(AYK_ACT_NONE, false, args.out_bf16);
+  args.mode = epilogue_mode(act, false, args.out_bf16);
   args.box_m = BM;
   args.m_tiles = M / BM;
   args.n_tiles = (N + BN - 1) / BN;

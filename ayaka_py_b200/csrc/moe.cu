@@ -9,12 +9,18 @@
 //
 // An expert's activation: g = min(gate, limit), u = clamp(up, -limit, limit),
 // y = g * sigmoid(slope * g) * (u + plus).  An infinite limit clamps nothing; slope 1 and plus 0 make it
-// silu(gate) * up.
+// silu(gate) * up.  Experts without a gate (a plain product with an activation of common.cuh in its epilogue) run
+// through the same kernels.
 //
 // Routing by sigmoid scores in groups (moe_route_scored_kernel): s = sigmoid(z); experts are ranked by
 // s + correction[e]; the experts are ``groups`` equal runs of consecutive experts, a run's score is the sum of its
 // two largest ranking scores, and only experts of the ``keep`` best runs can be chosen; the weights are
 // the chosen s divided by their sum, times a factor.
+//
+// The same kernel with softmax scores: s = softmax(z) over all experts; with a correction experts are ranked by
+// s + correction[e], without one by z itself (the same order, also where s underflows).  Two more things are
+// parameters of both: a run's score may be its largest ranking score alone, and the weights may be the chosen s as they are,
+// times the factor.
 #include <math.h>
 
 #include "common.cuh"
@@ -85,22 +91,37 @@ moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float
 // A warp per token.  Lane g holds the score of run g (at most 32 runs); the runs that may be chosen are a
 // bit mask that every lane holds; then the same repeated arg-max as above over the allowed experts' ranking
 // scores (the lower index wins a tie).
+template <bool SOFTMAX>
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits, long long stride,
-                        const float* __restrict__ correction, int T, int E, int top, int groups, int keep, float factor) {
+                        const float* __restrict__ correction, int T, int E, int top, int groups, int keep, int group_best,
+                        int normalize, float factor) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= T) return;
   const float* z = logits + (size_t)t * stride;
   const int per = E / groups;
+  float zmax = 0.f, inv_sum = 1.f;
+  if (SOFTMAX) {
+    float m = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+    zmax = warp_max(m);
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
+    inv_sum = 1.0f / warp_sum(sum);
+  }
+  auto score = [&](int e) { return SOFTMAX ? expf(z[e] - zmax) * inv_sum : sigmoidf(z[e]); };
+  auto ranking = [&](int e) {
+    if (SOFTMAX && !correction) return z[e];
+    return score(e) + (correction ? correction[e] : 0.f);
+  };
   unsigned allowed = 0xffffffffu;
   if (keep < groups) {
-    float mine = -INFINITY;                    // lane g: the sum of run g's two largest ranking scores
+    float mine = -INFINITY;                    // lane g: run g's largest ranking score, or the sum of its two largest
     for (int g = 0; g < groups; ++g) {
       float best = -INFINITY, second = -INFINITY;
       for (int e = g * per + lane; e < (g + 1) * per; e += 32) {
-        const float v = sigmoidf(z[e]) + (correction ? correction[e] : 0.f);
+        const float v = ranking(e);
         if (v > best) { second = best; best = v; } else if (v > second) second = v;
       }
 #pragma unroll
@@ -110,8 +131,8 @@ moe_route_scored_kernel(int* __restrict__ ids, float* __restrict__ weights, cons
         second = fmaxf(lo, fmaxf(second, os));
         best = hi;
       }
-      const float score = per > 1 ? best + second : best;
-      if (lane == g) mine = score;
+      const float total = (group_best == 2 && per > 1) ? best + second : best;
+      if (lane == g) mine = total;
     }
     int rank = 0;                              // runs that come before mine: a larger score, or the same and a lower index
     for (int g = 0; g < groups; ++g) {
@@ -125,25 +146,23 @@ moe_route_scored_kernel(int* __restrict__ ids, float* __restrict__ weights, cons
 #pragma unroll
   for (int k = 0; k < MAX_TOP; ++k) {
     if (k >= top) break;
-    float best = -INFINITY, best_s = 0.f;
+    float best = -INFINITY;
     int at = 0x7fffffff;
     for (int e = lane; e < E; e += 32) {
       bool taken = !((allowed >> (e / per)) & 1u);
 #pragma unroll
       for (int j = 0; j < MAX_TOP; ++j) taken |= (j < k && chosen[j] == e);
-      const float sc = sigmoidf(z[e]);
-      const float v = sc + (correction ? correction[e] : 0.f);
-      if (!taken && (v > best || (v == best && e < at) || at == 0x7fffffff)) { best = v; at = e; best_s = sc; }
+      const float v = ranking(e);
+      if (!taken && (v > best || (v == best && e < at) || at == 0x7fffffff)) { best = v; at = e; }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const float osc = __shfl_xor_sync(0xffffffffu, best_s, o);
       const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-      if (oa != 0x7fffffff && (at == 0x7fffffff || ob > best || (ob == best && oa < at))) { best = ob; at = oa; best_s = osc; }
+      if (oa != 0x7fffffff && (at == 0x7fffffff || ob > best || (ob == best && oa < at))) { best = ob; at = oa; }
     }
     chosen[k] = at;
-    value[k] = best_s;
+    value[k] = score(at);
   }
   if (lane == 0) {
     float sum = 0.f;
@@ -152,7 +171,7 @@ moe_route_scored_kernel(int* __restrict__ ids, float* __restrict__ weights, cons
       if (k >= top) break;
       sum += value[k];
     }
-    const float inv = factor / (sum + 1e-20f);
+    const float inv = normalize ? factor / (sum + 1e-20f) : factor;
 #pragma unroll
     for (int k = 0; k < MAX_TOP; ++k) {
       if (k >= top) break;
@@ -260,7 +279,7 @@ template <typename T, typename O, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(O* __restrict__ out, const T* __restrict__ a, long long a_stride, const T* __restrict__ w,
                 const int* __restrict__ sorted, const int* __restrict__ tiles, int top, int gather, int scatter, int N,
-                int N_w, int Kd, float limit, float slope, float plus) {
+                int N_w, int Kd, float limit, float slope, float plus, int act) {
   __shared__ float As[BK][TILE_ROWS + 1];
   __shared__ float Bs[GLU ? 2 : 1][BK][BN + 1];
   __shared__ int a_row[TILE_ROWS], o_row[TILE_ROWS];
@@ -328,7 +347,7 @@ moe_gemm_kernel(O* __restrict__ out, const T* __restrict__ a, long long a_stride
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= N) continue;
-      const float v = GLU ? glu_limited(acc[0][i][j], acc[GLU ? 1 : 0][i][j], limit, slope, plus) : acc[0][i][j];
+      const float v = GLU ? glu_limited(acc[0][i][j], acc[GLU ? 1 : 0][i][j], limit, slope, plus) : apply_activation(acc[0][i][j], act);
       out[(size_t)dst * N + n] = from_float<O>(v);
     }
   }
@@ -352,7 +371,7 @@ template <typename O, bool GLU>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long long a_stride,
                     const __nv_bfloat16* __restrict__ w, const int* __restrict__ sorted, const int* __restrict__ tiles,
-                    int top, int gather, int scatter, int N, int N_w, int Kd, float limit, float slope, float plus) {
+                    int top, int gather, int scatter, int N, int N_w, int Kd, float limit, float slope, float plus, int act) {
   __shared__ __align__(16) __nv_bfloat16 As[TILE_ROWS][TLD];
   __shared__ __align__(16) __nv_bfloat16 Bs[GLU ? 2 : 1][BN][TLD];
   __shared__ int a_row[TILE_ROWS], o_row[TILE_ROWS];
@@ -438,7 +457,7 @@ moe_gemm_mma_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, lo
           const int n = n0 + warp * 16 + j * 8 + tig * 2 + c;
           if (n >= N) continue;
           const float v0 = acc[0][i][j][half * 2 + c];
-          const float v = GLU ? glu_limited(v0, acc[GLU ? 1 : 0][i][j][half * 2 + c], limit, slope, plus) : v0;
+          const float v = GLU ? glu_limited(v0, acc[GLU ? 1 : 0][i][j][half * 2 + c], limit, slope, plus) : apply_activation(v0, act);
           out[(size_t)dst * N + n] = from_float<O>(v);
         }
     }
@@ -468,8 +487,8 @@ template <typename O, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long long a_stride,
                 const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids, int top, int gather, int N, int N_w,
-                int Kd, float limit, float slope, float plus) {
-  extern __shared__ __align__(16) float act[];          // [Kd]
+                int Kd, float limit, float slope, float plus, int act) {
+  extern __shared__ __align__(16) float xs[];          // [Kd]
   pdl_trigger();
   pdl_wait();
   const int pair = blockIdx.x;
@@ -482,8 +501,8 @@ moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long l
     lo.z = __uint_as_float(v.y << 16); lo.w = __uint_as_float(v.y & 0xffff0000u);
     hi.x = __uint_as_float(v.z << 16); hi.y = __uint_as_float(v.z & 0xffff0000u);
     hi.z = __uint_as_float(v.w << 16); hi.w = __uint_as_float(v.w & 0xffff0000u);
-    *reinterpret_cast<float4*>(act + i * 8) = lo;
-    *reinterpret_cast<float4*>(act + i * 8 + 4) = hi;
+    *reinterpret_cast<float4*>(xs + i * 8) = lo;
+    *reinterpret_cast<float4*>(xs + i * 8 + 4) = hi;
   }
   __syncthreads();
   const __nv_bfloat16* we = w + (size_t)ids[pair] * N_w * Kd;
@@ -497,7 +516,7 @@ moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long l
     const __nv_bfloat16* r0 = we + (size_t)n0 * Kd;
     const __nv_bfloat16* r1 = we + (size_t)(two ? n1 : n0) * Kd;
     for (int k = lane * 8; k < Kd; k += 256) {
-      const float4 x0 = *reinterpret_cast<const float4*>(act + k), x1 = *reinterpret_cast<const float4*>(act + k + 4);
+      const float4 x0 = *reinterpret_cast<const float4*>(xs + k), x1 = *reinterpret_cast<const float4*>(xs + k + 4);
       const uint4 wa = *reinterpret_cast<const uint4*>(r0 + k), wb = *reinterpret_cast<const uint4*>(r1 + k);
       if (GLU) {
         const uint4 wc = *reinterpret_cast<const uint4*>(r0 + (size_t)N * Kd + k), wd = *reinterpret_cast<const uint4*>(r1 + (size_t)N * Kd + k);
@@ -510,8 +529,8 @@ moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long l
     g0 = warp_sum(g0); g1 = warp_sum(g1);
     if (GLU) { u0 = warp_sum(u0); u1 = warp_sum(u1); }
     if (lane == 0) {
-      out[(size_t)pair * N + n0] = from_float<O>(GLU ? glu_limited(g0, u0, limit, slope, plus) : g0);
-      if (two) out[(size_t)pair * N + n1] = from_float<O>(GLU ? glu_limited(g1, u1, limit, slope, plus) : g1);
+      out[(size_t)pair * N + n0] = from_float<O>(GLU ? glu_limited(g0, u0, limit, slope, plus) : apply_activation(g0, act));
+      if (two) out[(size_t)pair * N + n1] = from_float<O>(GLU ? glu_limited(g1, u1, limit, slope, plus) : apply_activation(g1, act));
     }
   }
 }
@@ -563,36 +582,39 @@ AYK_EXPORT int ayk_moe_route(int* ids, float* weights, int* sorted, int* tiles, 
   return ayk_check_launch("ayk_moe_route");
 }
 
-// The same plan after routing by sigmoid scores in groups (see the head of the file).  correction [E] float32
-// or null; groups equal runs of consecutive experts (at most 32) of which keep may be chosen from.
+// The same plan after routing by sigmoid (or, with ``softmax``, softmax) scores in groups (see the head of the file).
+// correction [E] float32 or null; groups equal runs of consecutive experts (at most 32) of which keep may be chosen from;
+// group_best: 1 or 2 scores of a run make its own; normalize: the weights are divided by their sum.
 AYK_EXPORT int ayk_moe_route_scored(int* ids, float* weights, int* sorted, int* tiles, const float* logits, long long stride,
                                     const float* correction, int T, int E, int top, int groups, int keep, float factor,
-                                    cudaStream_t stream) {
+                                    int softmax, int group_best, int normalize, cudaStream_t stream) {
   if (T == 0) return 0;
   AYK_REQUIRE(top >= 1 && top <= MAX_TOP && top <= E, "ayk_moe_route_scored: top %d of %d experts (at most %d)", top, E, MAX_TOP);
   AYK_REQUIRE(E <= 4096, "ayk_moe_route_scored: %d experts (at most 4096)", E);
   AYK_REQUIRE(groups >= 1 && groups <= 32 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top,
               "ayk_moe_route_scored: %d experts in %d groups of which %d are kept cannot give %d choices", E, groups, keep, top);
-  ayk_launch(moe_route_scored_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, ids, weights, logits, stride, correction, T, E,
-             top, groups, keep, factor);
+  AYK_REQUIRE(group_best == 1 || group_best == 2, "ayk_moe_route_scored: a group's score is its best or its two best");
+  ayk_launch(softmax ? moe_route_scored_kernel<true> : moe_route_scored_kernel<false>, dim3((T + 3) / 4), dim3(128), 0, stream, ids,
+             weights, logits, stride, correction, T, E, top, groups, keep, group_best, normalize, factor);
   ayk_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, sorted, tiles, (const int*)ids,
              T * top, E);
   return ayk_check_launch("ayk_moe_route_scored");
 }
 
-// See moe_gemm_kernel.  dtype: of a and w; out_dtype: of out (the activation's rows may be bfloat16,
-// plain products are float32).  max_tiles: the grid's first dimension.
+// See moe_gemm_kernel.  dtype: of a and w; out_dtype: of out (gated rows are of the operands' dtype, plain
+// products, with the activation ``act``, of that or float32).  max_tiles: the grid's first dimension.
 AYK_EXPORT int ayk_moe_gemm(void* out, const void* a, long long a_stride, const void* w, const int* sorted,
                             const int* tiles, int max_tiles, int top, int gather, int scatter, int N, int N_w, int Kd,
-                            int glu, float limit, float slope, float plus, int dtype, int out_dtype, cudaStream_t stream) {
+                            int glu, float limit, float slope, float plus, int act, int dtype, int out_dtype,
+                            cudaStream_t stream) {
   if (max_tiles == 0 || N == 0) return 0;
   dim3 grid(max_tiles, (N + BN - 1) / BN);
 #define AYK_MOE(T, O, G)                                                                                              \
   ayk_launch(moe_gemm_kernel<T, O, G>, grid, dim3(256), 0, stream, (O*)out, (const T*)a, a_stride, (const T*)w, sorted, \
-             tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus)
+             tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus, act)
 #define AYK_MOE_MMA(O, G)                                                                                        \
   ayk_launch(moe_gemm_mma_kernel<O, G>, grid, dim3(128), 0, stream, (O*)out, (const __nv_bfloat16*)a, a_stride, \
-             (const __nv_bfloat16*)w, sorted, tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus)
+             (const __nv_bfloat16*)w, sorted, tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus, act)
   if (dtype == AYK_DTYPE_F32) {
     AYK_REQUIRE(out_dtype == AYK_DTYPE_F32, "ayk_moe_gemm: float32 operands give float32 rows");
     if (glu) AYK_MOE(float, float, true); else AYK_MOE(float, float, false);
@@ -601,8 +623,10 @@ AYK_EXPORT int ayk_moe_gemm(void* out, const void* a, long long a_stride, const 
     if (glu) {
       AYK_REQUIRE(out_dtype == AYK_DTYPE_BF16, "ayk_moe_gemm: the activation's rows are bfloat16 here");
       if (tensor) AYK_MOE_MMA(__nv_bfloat16, true); else AYK_MOE(__nv_bfloat16, __nv_bfloat16, true);
+    } else if (out_dtype == AYK_DTYPE_BF16) {
+      if (tensor) AYK_MOE_MMA(__nv_bfloat16, false); else AYK_MOE(__nv_bfloat16, __nv_bfloat16, false);
     } else {
-      AYK_REQUIRE(out_dtype == AYK_DTYPE_F32, "ayk_moe_gemm: plain products give float32 rows");
+      AYK_REQUIRE(out_dtype == AYK_DTYPE_F32, "ayk_moe_gemm: unknown dtype %d", out_dtype);
       if (tensor) AYK_MOE_MMA(float, false); else AYK_MOE(__nv_bfloat16, float, false);
     }
   } else {
@@ -653,21 +677,25 @@ AYK_EXPORT int ayk_moe_combine(float* shared, const float* picked, const int* ro
 }
 
 // The products of a few pairs, pair by pair (see moe_gemv_kernel): bfloat16 a and w, K a multiple of 8 and at most
-// 12,288.  glu: out [pairs, N] bfloat16 = activation of (gate, up) rows of w [E, 2 N, K], a row p / top; else
-// out [pairs, N] float32 = a row p times w [E, N, K].
+// 12,288.  gather: pair p reads row p / top of a, else row p.  glu: out [pairs, N] bfloat16 = activation of (gate, up)
+// rows of w [E, 2 N, K]; else out [pairs, N] (out_dtype) = act(row times w [E, N, K]).
 AYK_EXPORT int ayk_moe_gemv_takes(int Kd, long long a_stride) { return Kd % 8 == 0 && a_stride % 8 == 0 && Kd <= 12288; }
 
 AYK_EXPORT int ayk_moe_gemv(void* out, const void* a, long long a_stride, const void* w, const int* ids, int pairs, int top,
-                            int N, int N_w, int Kd, int glu, float limit, float slope, float plus, cudaStream_t stream) {
+                            int N, int N_w, int Kd, int gather, int glu, float limit, float slope, float plus, int act, int out_dtype,
+                            cudaStream_t stream) {
   if (pairs == 0 || N == 0) return 0;
   AYK_REQUIRE(ayk_moe_gemv_takes(Kd, a_stride), "ayk_moe_gemv: rows of %d elements (stride %lld)", Kd, a_stride);
   dim3 grid(pairs, (N + GV_COLS - 1) / GV_COLS);
   const size_t smem = (size_t)Kd * sizeof(float);
   if (glu)
     ayk_launch(moe_gemv_kernel<__nv_bfloat16, true>, grid, dim3(256), smem, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)a,
-               a_stride, (const __nv_bfloat16*)w, ids, top, 1, N, N_w, Kd, limit, slope, plus);
+               a_stride, (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act);
+  else if (out_dtype == AYK_DTYPE_BF16)
+    ayk_launch(moe_gemv_kernel<__nv_bfloat16, false>, grid, dim3(256), smem, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)a,
+               a_stride, (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act);
   else
     ayk_launch(moe_gemv_kernel<float, false>, grid, dim3(256), smem, stream, (float*)out, (const __nv_bfloat16*)a, a_stride,
-               (const __nv_bfloat16*)w, ids, top, 0, N, N_w, Kd, limit, slope, plus);
+               (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act);
   return ayk_check_launch("ayk_moe_gemv");
 }

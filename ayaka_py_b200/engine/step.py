@@ -66,6 +66,11 @@ class StepContext:
     # of the step's inputs (or a graph launch) lies between.  Kernels may read them ahead of the
     # kernels launched just before them.
     earlier_rows_settled: bool = False
+    # What one part of a step leaves for a later one, by a name that both know (the values of an earlier layer) or by
+    # the part that left it; emptied at the start of a forward.
+    carry: dict = field(default_factory=dict)
+    # The norm that opens the next run step, for a block whose last kernel can make it (``carry["opened"]``); None: there is none.
+    following: object = None
 
 
 class StepRunner:

@@ -132,12 +132,17 @@ class Model:
         """One step.  Returns logits [S, V] float32 at ``ctx.want_rows``."""
         if not self.loaded:
             raise RuntimeError("the model has no weights yet")
+        ctx.carry.clear()
         x = self.embedding.forward(ctx, self.position)
         x0 = x.clone() if any(step.add_input for step in self.spec.order) else None     # the blocks write the stream in place
-        for step, caches in zip(self.spec.order, self.bindings):
+        order = self.spec.order
+        for i, (step, caches) in enumerate(zip(order, self.bindings)):
             if step.add_input:
                 x = ops.add_(x, x0)
+            after = order[i + 1] if i + 1 < len(order) else None
+            ctx.following = self.blocks[after.layer].opening_norm() if after is not None and not after.add_input else None
             x = self.blocks[step.layer].forward(x, ctx, caches)
+        ctx.carry.clear()
         if ctx.num_wanted == 0:
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=x.device)
         h = self.final_norm.forward(x, ctx, rows=ctx.want_rows)

@@ -825,7 +825,7 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
                       key_heads: int, key_dim: int, scale: float, slopes: torch.Tensor | None = None,
                       window: int | None = None, keep_first: int = 0, gate: torch.Tensor | None = None,
                       maps: int = 1, lam: float = 0.0, post_scale: float = 1.0, eps: float = 0.0,
-                      tensor_cores: bool = True, chunk: int | None = None) -> torch.Tensor:
+                      tensor_cores: bool = True, chunk: int | None = None, sinks: torch.Tensor | None = None) -> torch.Tensor:
     """Softmax attention of the step's rows over the paged cache with keys and values grouped separately:
     ``heads`` query heads of ``key_dim`` read ``key_heads`` key heads (the pages' rows taken as
     [key_heads, key_dim]) and the value heads of ``vpages``; score (q . k) scale - slopes[h] (i - j); key j
@@ -834,7 +834,9 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
     sigmoid(gate).  ``maps`` == 2: the query heads are [group][map][head of the group] and the result is per
     head o1 - lam o2, divided by its root mean square (``eps`` under the root), times ``post_scale``; a
     gate then has one number per output head.  When every request brings one row the context is cut into parts that a
-    second kernel merges.  Returns [T, heads / maps * vdim] of the pages' dtype."""
+    second kernel merges (with a window that keeps no first keys, the parts that a window can reach).  ``sinks``
+    float32 [heads]: exp(sinks[h]) more in every denominator (a key that is always seen and has no value).
+    Returns [T, heads / maps * vdim] of the pages' dtype."""
     lib = _ready()
     lib.ayk_grouped_attention_tensor_cores(ctypes.c_int(1 if tensor_cores else 0))
     pages, P, VH, DV = vpages.shape
@@ -850,8 +852,16 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
                              gate.shape[1] < (heads * DV if maps == 1 else out_heads)):
         raise KernelError("grouped_attention: the gate is float32 rows as wide as the output (one number per head with two maps)")
     out = torch.empty((T, out_heads * DV), dtype=q.dtype, device=q.device)
-    part_keys = grouped_part(ctx.cache.max_len)
-    parts = max(1, -(-ctx.cache.max_len // part_keys)) if ctx.max_q_len == 1 else 1
+    if sinks is not None and _f32(sinks, "sinks").numel() != heads:
+        raise KernelError("grouped_attention: one sink per query head")
+    span, from_window = ctx.cache.max_len, False
+    part_keys = grouped_part(span)
+    parts = max(1, -(-span // part_keys)) if ctx.max_q_len == 1 else 1
+    if parts > 1 and window and not keep_first and not chunk and window < span:
+        # a row reads its window only: the parts from the one that holds the window's first key on
+        part_keys = grouped_part(window)
+        parts = -(-(window - 1) // part_keys) + 1
+        from_window = parts > 1
     two_steps = parts > 1 or maps > 1
     po = pml = None
     if two_steps:
@@ -862,17 +872,168 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
                                       _ptr(_i32(table, "table")), ctypes.c_int(table.stride(0)), _ptr(ctx.req_q_start),
                                       _ptr(ctx.req_pos0), ctypes.c_int(ctx.num_requests), ctypes.c_int(T), ctypes.c_int(heads),
                                       ctypes.c_int(key_heads), ctypes.c_int(VH), ctypes.c_int(key_dim), ctypes.c_int(DV),
-                                      ctypes.c_int(P), ctypes.c_float(scale), _ptr(slopes), ctypes.c_int(window or 0),
+                                      ctypes.c_int(P), ctypes.c_float(scale), _ptr(slopes), _ptr(sinks), ctypes.c_int(window or 0),
                                       ctypes.c_int(keep_first), ctypes.c_int(chunk or 0), _ptr(None if two_steps else gate),
                                       ctypes.c_longlong(gate_stride),
-                                      ctypes.c_int(parts), ctypes.c_int(part_keys), ctypes.c_int(_tag(q.dtype)), _stream()))
+                                      ctypes.c_int(parts), ctypes.c_int(part_keys), ctypes.c_int(1 if from_window else 0),
+                                      ctypes.c_int(_tag(q.dtype)), _stream()))
     if two_steps:
         _launch(lib.ayk_grouped_finish(_ptr(out), _ptr(po), _ptr(pml), _ptr(ctx.positions), ctypes.c_int(T), ctypes.c_int(heads),
-                                       ctypes.c_int(DV), ctypes.c_int(parts), ctypes.c_int(part_keys), ctypes.c_int(maps),
+                                       ctypes.c_int(DV), ctypes.c_int(parts), ctypes.c_int(part_keys),
+                                       ctypes.c_int(window if from_window else 0), ctypes.c_int(maps),
                                        ctypes.c_int(hpg if maps > 1 else 1), _ptr(gate), ctypes.c_longlong(gate_stride),
                                        ctypes.c_float(lam), ctypes.c_float(post_scale), ctypes.c_float(eps),
                                        ctypes.c_int(_tag(q.dtype)), _stream()))
     return out
+
+
+def rotary_prepare(proj: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tensor, freq: torch.Tensor | None, rot_dims: int, ctx,
+                   table: torch.Tensor, heads: int, writes: bool, out_dtype: torch.dtype, first: torch.Tensor | None = None,
+                   mix: float = 0.0) -> torch.Tensor:
+    """From float32 projection rows [q | k | v | ...]: the first ``rot_dims`` dimensions of every query and key head
+    rotated by the position (dimension i with i + rot_dims/2; 0: none), keys and values into their pages (unless
+    ``writes`` is False), the queries returned [T, heads * dim] in ``out_dtype``.  ``first``: float32 rows as wide as a
+    token's values; the values filed are (1 - mix) v + mix first."""
+    lib = _ready()
+    _f32(proj, "proj")
+    T = proj.shape[0]
+    pages, P, G, D = kpages.shape
+    v_width = vpages.shape[2] * vpages.shape[3]
+    if (proj.shape[1] < (heads + G) * D + v_width or kpages.dtype != out_dtype or vpages.dtype != out_dtype
+            or not kpages.is_contiguous() or not vpages.is_contiguous() or rot_dims > D
+            or (rot_dims and _f32(freq, "freq").numel() * 2 != rot_dims)):
+        raise KernelError("rotary_prepare: projection rows, frequencies or pages do not fit")
+    if first is not None and (first.dtype != torch.float32 or first.shape != (T, v_width) or first.stride(1) != 1):
+        raise KernelError("rotary_prepare: the values to mix in must be float32 rows as wide as a token's values")
+    q = torch.empty((T, heads * D), dtype=out_dtype, device=proj.device)
+    _launch(lib.ayk_rotary_prepare(_ptr(q), _ptr(kpages), _ptr(vpages), _ptr(proj), ctypes.c_longlong(proj.stride(0)),
+                                   _ptr(freq if rot_dims else None), ctypes.c_int(rot_dims), _ptr(first),
+                                   ctypes.c_longlong(first.stride(0) if first is not None else 0), ctypes.c_float(1.0 - mix),
+                                   ctypes.c_float(mix), _ptr(ctx.row_req), _ptr(ctx.positions), _ptr(_i32(table, "table")),
+                                   ctypes.c_int(table.stride(0)), ctypes.c_int(P), ctypes.c_int(T), ctypes.c_int(heads), ctypes.c_int(G),
+                                   ctypes.c_int(D), ctypes.c_int(v_width), ctypes.c_int(1 if writes else 0),
+                                   ctypes.c_int(_tag(out_dtype)), _stream()))
+    return q
+
+
+DECAY_CHUNK = 64          # tokens that the chunked form of the decayed recurrence takes at a time
+
+
+def decay_chunk_takes(dim: int) -> bool:
+    """Whether the chunked (bfloat16, tensor-core) form of the decayed recurrence takes heads of ``dim`` numbers."""
+    return bool(library().ayk_decay_chunk_takes(ctypes.c_int(dim)))
+
+
+def decay_recurrence(rows: torch.Tensor, state: torch.Tensor, powers: torch.Tensor, ctx, heads: int, dim: int, vdim: int,
+                     slice_cols: int = 0) -> torch.Tensor:
+    """S <- lambda_h S + k v^T, o = S^T q per head over the step's rows, request by request, from and into ``state``
+    [slots, heads, dim, vdim] float32; returns o [T, heads * vdim] float32.  ``powers`` float32 [heads, 65]:
+    lambda_h^n.  float32 ``rows`` [q | k | v | ...] before their SiLU: token by token; bfloat16 rows
+    [silu q | silu k | silu v]: 64 tokens at a time on the tensor cores (``slice_cols``: value columns per block, 16 or
+    32; 0: chosen by the grid)."""
+    lib = _ready()
+    _f32(state, "state"); _f32(powers, "powers")
+    T = rows.shape[0]
+    if (rows.stride(1) != 1 or rows.shape[1] < heads * (2 * dim + vdim) or state.shape[1:] != (heads, dim, vdim)
+            or powers.shape != (heads, DECAY_CHUNK + 1)):
+        raise KernelError("decay_recurrence: rows, state or powers do not fit")
+    out = torch.empty((T, heads * vdim), dtype=torch.float32, device=rows.device)
+    common = (_ptr(out), _ptr(state), _ptr(rows), ctypes.c_longlong(rows.stride(0)), _ptr(powers), _ptr(ctx.req_q_start),
+              _ptr(ctx.req_slot), ctypes.c_int(ctx.num_requests), ctypes.c_int(heads), ctypes.c_int(dim), ctypes.c_int(vdim))
+    settled = ctypes.c_int(1 if getattr(ctx, "earlier_rows_settled", False) else 0)
+    if rows.dtype == torch.bfloat16:
+        _launch(lib.ayk_decay_chunk(*common, ctypes.c_int(slice_cols), settled, _stream()))
+    elif rows.dtype == torch.float32:
+        _launch(lib.ayk_decay_walk(*common, settled, _stream()))
+    else:
+        raise KernelError(f"decay_recurrence: rows of {rows.dtype}")
+    return out
+
+
+def rmsnorm_gated(raw: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """raw / sqrt(mean(raw^2) + eps) * weight * sigmoid(gate) over whole rows; float32 in, 32-bit arithmetic."""
+    lib = _ready()
+    _f32(raw, "raw"); _f32(weight, "weight")
+    T, n = raw.shape
+    if gate.dtype != torch.float32 or gate.shape != (T, n) or gate.stride(1) != 1 or weight.numel() != n:
+        raise KernelError("rmsnorm_gated: gate rows or weight do not fit")
+    out = torch.empty((T, n), dtype=out_dtype, device=raw.device)
+    _launch(lib.ayk_decay_finish(_ptr(out), _ptr(raw), _ptr(gate), ctypes.c_longlong(gate.stride(0)), _ptr(weight), ctypes.c_int(T),
+                                 ctypes.c_int(n), ctypes.c_float(eps), ctypes.c_int(_tag(out_dtype)), _stream()))
+    return out
+
+
+class PickedRows:
+    """A routed feed-forward's result before its sum: float32 rows of the (token, choice) pairs, their weights and
+    where each pair's row lies (None: in order).  ``stream_update`` adds them up on the way."""
+
+    def __init__(self, rows: torch.Tensor, route: "MoeRoute", row_of_pair: torch.Tensor | None):
+        self.rows, self.route, self.row_of_pair = rows, route, row_of_pair
+
+
+_STREAM_POST = {"none": 0, "copy": 1, "layernorm": 2, "rmsnorm": 3}
+
+
+def stream_update(x: torch.Tensor, y: "torch.Tensor | PickedRows", scale: torch.Tensor, gate: torch.Tensor | None = None,
+                  eps: float = 0.0, post: str = "none", next_weight: torch.Tensor | None = None, next_bias: torch.Tensor | None = None,
+                  next_eps: float = 0.0, out_dtype: torch.dtype = torch.float32) -> torch.Tensor | None:
+    """x += y * scale * sigmoid(gate) with ``gate`` (float32 rows [T, d]), or x += rmsnorm(y) * scale without, in place on
+    the float32 residual stream.  ``post``: what the same kernel returns of the updated rows in ``out_dtype``:
+    nothing, a copy, their layer norm or their RMS norm with ``next_weight``."""
+    lib = _ready()
+    _f32(x, "x"); _f32(scale, "scale")
+    T, d = x.shape
+    picked = row_of_pair = weights = None
+    top = 0
+    if isinstance(y, PickedRows):
+        picked, row_of_pair, weights, top = _f32(y.rows, "picked"), y.row_of_pair, y.route.weights, y.route.top
+        if picked.shape[1] != d or weights.shape[0] != T or (row_of_pair is None and picked.shape[0] != T * top):
+            raise KernelError("stream_update: the pairs' rows do not fit the stream")
+        y = None
+    elif _f32(y, "y").shape != x.shape:
+        raise KernelError("stream_update: y must have the stream's shape")
+    if scale.numel() != d or (gate is not None and (gate.dtype != torch.float32 or gate.shape != (T, d) or gate.stride(1) != 1)):
+        raise KernelError("stream_update: scale or gate rows do not fit")
+    if post in ("layernorm", "rmsnorm") and _f32(next_weight, "next_weight").numel() != d:
+        raise KernelError("stream_update: the following norm's weight does not fit")
+    out = torch.empty((T, d), dtype=out_dtype, device=x.device) if post != "none" else None
+    _launch(lib.ayk_stream_update(_ptr(x), _ptr(out), _ptr(y), _ptr(picked), _ptr(row_of_pair), _ptr(weights), ctypes.c_int(top),
+                                  _ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(scale),
+                                  _ptr(next_weight), _ptr(next_bias), ctypes.c_int(T), ctypes.c_int(d),
+                                  ctypes.c_int(0 if gate is not None else 1), ctypes.c_int(_STREAM_POST[post]), ctypes.c_float(eps),
+                                  ctypes.c_float(next_eps), ctypes.c_int(_tag(out_dtype)), _stream()))
+    return out
+
+
+TOKEN_GATE_ROWS = 64      # up to this many rows the token gate's product runs a warp per number, straight from the stream
+
+
+def token_gate(tokens: torch.Tensor, table: torch.Tensor, col0: int, n: int, x: torch.Tensor | None = None,
+               weight: torch.Tensor | None = None, z: torch.Tensor | None = None) -> torch.Tensor:
+    """gelu_tanh(x @ weight^T) * table[tokens, col0 .. col0 + n), in the table's dtype: from the float32 stream and
+    ``weight`` [n, d], or from the product ``z`` (float32 [T, n]) already made."""
+    lib = _ready()
+    T = tokens.numel()
+    if not table.is_contiguous() or col0 + n > table.shape[1]:
+        raise KernelError("token_gate: the table's columns do not fit")
+    if z is not None:
+        if _f32(z, "z").shape != (T, n):
+            raise KernelError("token_gate: z must be [T, n]")
+    elif _f32(x, "x").shape[0] != T or weight.shape != (n, x.shape[1]) or weight.dtype != table.dtype or not weight.is_contiguous():
+        raise KernelError("token_gate: stream and matrix do not fit")
+    out = torch.empty((T, n), dtype=table.dtype, device=table.device)
+    _launch(lib.ayk_token_gate(_ptr(out), _ptr(x if z is None else None), _ptr(weight if z is None else None), _ptr(z), _ptr(table),
+                               ctypes.c_longlong(table.stride(0)), ctypes.c_int(col0), _ptr(_i32(tokens, "tokens")), ctypes.c_int(T),
+                               ctypes.c_int(x.shape[1] if z is None else 0), ctypes.c_int(n), ctypes.c_int(_tag(table.dtype)), _stream()))
+    return out
+
+
+def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x = cap * tanh(x / cap), in place (contiguous float32)."""
+    lib = _ready()
+    _f32(x, "x")
+    _launch(lib.ayk_softcap(_ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(cap), _stream()))
+    return x
 
 
 class MoeRoute:
@@ -886,10 +1047,12 @@ class MoeRoute:
 
 def moe_route(logits: torch.Tensor, experts: int, top: int, scored: dict | None = None) -> MoeRoute:
     """The ``top`` largest of each row's first ``experts`` float32 logits, weighted by the softmax over
-    the chosen ones, and the plan of the grouped products.  ``scored`` = {correction, groups, keep, factor}:
-    routing by sigmoid scores s instead; experts are ranked by s + correction (float32 [experts] or None) among
-    the experts of the ``keep`` best of ``groups`` equal runs of consecutive experts (a run's score: the sum of its two
-    largest ranking scores), the weights are the chosen s over their sum, times ``factor``."""
+    the chosen ones, and the plan of the grouped products.  ``scored`` = {correction, groups, keep, factor, scores,
+    group_best, normalize}: routing by scores s of all experts instead, sigmoid (the default) or ``scores`` "softmax";
+    experts are ranked by s + correction (float32 [experts] or None) among the experts of the ``keep`` best of
+    ``groups`` equal runs of consecutive experts (a run's score: the sum of its two largest ranking scores, or with
+    ``group_best`` 1 the largest); the weights are the chosen s over their sum (``normalize`` False: as they are),
+    times ``factor``."""
     lib = _ready()
     if logits.dtype != torch.float32 or logits.stride(1) != 1 or logits.shape[1] < experts:
         raise KernelError("moe_route: logits must be float32 rows of at least ``experts`` columns")
@@ -908,7 +1071,9 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, scored: dict | None 
                                          ctypes.c_longlong(logits.stride(0)), _ptr(correction), ctypes.c_int(T),
                                          ctypes.c_int(experts), ctypes.c_int(top), ctypes.c_int(int(scored.get("groups", 1))),
                                          ctypes.c_int(int(scored.get("keep", 1))), ctypes.c_float(float(scored.get("factor", 1.0))),
-                                         _stream()))
+                                         ctypes.c_int(1 if scored.get("scores", "sigmoid") == "softmax" else 0),
+                                         ctypes.c_int(int(scored.get("group_best", 2))),
+                                         ctypes.c_int(1 if scored.get("normalize", True) else 0), _stream()))
     else:
         _launch(lib.ayk_moe_route(_ptr(ids), _ptr(weights), _ptr(sorted_pairs), _ptr(tiles), _ptr(logits),
                                   ctypes.c_longlong(logits.stride(0)), ctypes.c_int(T), ctypes.c_int(experts), ctypes.c_int(top), _stream()))
@@ -925,25 +1090,29 @@ def _glu(glu: tuple | None) -> tuple[float, float, float]:
     return (float(glu[0]), float(glu[1]), float(glu[2]) if len(glu) > 2 else 1.0)
 
 
-def moe_gemm(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None, out_dtype: torch.dtype) -> torch.Tensor:
+def moe_gemm(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None, out_dtype: torch.dtype,
+             activation: str | None = None) -> torch.Tensor:
     """Grouped product over the sorted pairs.  ``glu`` = (limit, slope): a holds the tokens' rows
     [T, K], w [experts, 2 N, K] gate over up, and the result is the experts' activation
-    min(g, limit) sigmoid(slope g) (clamp(u) + 1) per sorted pair, [T * top, N] in ``out_dtype``.  ``glu`` None:
-    a holds rows per sorted pair, w [experts, N, K], and the float32 result [T * top, N] lies pair by pair
-    (token-major).  bfloat16 operands run on the tensor cores, float32 on the FP32 pipes."""
+    min(g, limit) sigmoid(slope g) (clamp(u) + 1) per sorted pair, [T * top, N] in ``out_dtype``.  ``activation``
+    instead: a holds the tokens' rows, w [experts, N, K], the result is the activation of the product, laid out
+    alike.  Neither: a holds rows per sorted pair, w [experts, N, K], and the float32 result [T * top, N] lies pair
+    by pair (token-major).  bfloat16 operands run on the tensor cores, float32 on the FP32 pipes."""
     lib = _ready()
     E, n_w, K = w.shape
-    if a.dtype != w.dtype or a.shape[1] != K or a.stride(1) != 1 or not w.is_contiguous():
+    if a.dtype != w.dtype or a.shape[1] != K or a.stride(1) != 1 or not w.is_contiguous() or (glu is not None and activation is not None):
         raise KernelError("moe_gemm: operands do not fit")
     pairs = route.sorted.numel()
     N = n_w // 2 if glu is not None else n_w
+    first = glu is not None or activation is not None
     out = torch.empty((pairs, N), dtype=out_dtype, device=a.device)
     limit, slope, plus = _glu(glu)
     _launch(lib.ayk_moe_gemm(_ptr(out), _ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), _ptr(route.sorted), _ptr(route.tiles),
-                             ctypes.c_int(route.max_tiles), ctypes.c_int(route.top), ctypes.c_int(1 if glu is not None else 0),
-                             ctypes.c_int(0 if glu is not None else 1), ctypes.c_int(N), ctypes.c_int(n_w), ctypes.c_int(K),
+                             ctypes.c_int(route.max_tiles), ctypes.c_int(route.top), ctypes.c_int(1 if first else 0),
+                             ctypes.c_int(0 if first else 1), ctypes.c_int(N), ctypes.c_int(n_w), ctypes.c_int(K),
                              ctypes.c_int(1 if glu is not None else 0), ctypes.c_float(limit), ctypes.c_float(slope),
-                             ctypes.c_float(plus), ctypes.c_int(_tag(a.dtype)), ctypes.c_int(_tag(out_dtype)), _stream()))
+                             ctypes.c_float(plus), ctypes.c_int(ACTIVATIONS[activation or "none"]), ctypes.c_int(_tag(a.dtype)),
+                             ctypes.c_int(_tag(out_dtype)), _stream()))
     return out
 
 
@@ -953,21 +1122,25 @@ def moe_gemv_takes(a: torch.Tensor, w: torch.Tensor) -> bool:
             and bool(_ready().ayk_moe_gemv_takes(ctypes.c_int(w.shape[2]), ctypes.c_longlong(a.stride(0)))))
 
 
-def moe_gemv(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None) -> torch.Tensor:
+def moe_gemv(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None, activation: str | None = None) -> torch.Tensor:
     """The experts' product for a handful of pairs, each pair streaming its expert's matrix on its own: no
     sorting, rows lie pair by pair (token-major).  ``glu`` = (limit, slope): a [T, K] tokens' rows, w
-    [experts, 2 N, K], bfloat16 activations [T * top, N]; None: a [T * top, K], w [experts, N, K], float32 out."""
+    [experts, 2 N, K], bfloat16 activations [T * top, N]; ``activation``: a [T, K], w [experts, N, K], bfloat16
+    activations of the product; neither: a [T * top, K], w [experts, N, K], float32 out."""
     lib = _ready()
     E, n_w, K = w.shape
     pairs = route.ids.numel()
     N = n_w // 2 if glu is not None else n_w
-    if a.shape[1] != K or a.stride(1) != 1 or not w.is_contiguous() or not moe_gemv_takes(a, w):
+    first = glu is not None or activation is not None
+    if a.shape[1] != K or a.stride(1) != 1 or not w.is_contiguous() or not moe_gemv_takes(a, w) or (glu is not None and activation is not None):
         raise KernelError("moe_gemv: operands do not fit")
-    out = torch.empty((pairs, N), dtype=torch.bfloat16 if glu is not None else torch.float32, device=a.device)
+    out_dtype = torch.bfloat16 if first else torch.float32
+    out = torch.empty((pairs, N), dtype=out_dtype, device=a.device)
     limit, slope, plus = _glu(glu)
     _launch(lib.ayk_moe_gemv(_ptr(out), _ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), _ptr(route.ids), ctypes.c_int(pairs),
-                             ctypes.c_int(route.top), ctypes.c_int(N), ctypes.c_int(n_w), ctypes.c_int(K),
-                             ctypes.c_int(1 if glu is not None else 0), ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(plus), _stream()))
+                             ctypes.c_int(route.top), ctypes.c_int(N), ctypes.c_int(n_w), ctypes.c_int(K), ctypes.c_int(1 if first else 0),
+                             ctypes.c_int(1 if glu is not None else 0), ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(plus),
+                             ctypes.c_int(ACTIVATIONS[activation or "none"]), ctypes.c_int(_tag(out_dtype)), _stream()))
     return out
 
 
@@ -987,15 +1160,16 @@ def glu_limited(x: torch.Tensor, n: int, limit: float, slope: float, out_dtype: 
 MOE_TENSOR_PAIRS = 64         # (token, choice) pairs from which the experts' products run on tcgen05
 
 
-def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.Tensor, route: MoeRoute, limit: float,
-                   slope: float, plus: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.Tensor, route: MoeRoute, limit: float = float("inf"),
+                   slope: float = 1.0, plus: float = 1.0, activation: str | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """The experts of a step on tcgen05 (bfloat16): the pairs' rows are gathered expert by expert, every expert's
     starting at a multiple of 128 rows, and the two products run as grouped forms of the many-row kernel, each
-    128-row tile against the matrix of its expert.  in_weight [experts, 2 inner, width] gate over up,
+    128-row tile against the matrix of its expert.  in_weight [experts, 2 inner, width] gate over up (or, with
+    ``activation``, [experts, inner, width] and that activation in the first product's epilogue),
     down_weight [experts, width, inner].  Returns (float32 rows [padded, width], row of every pair)."""
     lib = _ready()
     E, n1, d = in_weight.shape
-    inner = n1 // 2
+    inner = n1 if activation is not None else n1 // 2
     T = h.shape[0]
     pairs = T * route.top
     pad = int(lib.ayk_moe_pad_rows())
@@ -1011,13 +1185,14 @@ def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.
     launches += 1
     both = torch.empty((max_tiles * pad, n1), dtype=torch.bfloat16, device=dev_)
     _launch(lib.ayk_gemm_tc_prefill_grouped(_ptr(both), _ptr(gathered), _ptr(in_weight), _ptr(w_rows[0]), ctypes.c_int(max_tiles * pad),
-                                            ctypes.c_int(n1), ctypes.c_int(d), ctypes.c_int(E * n1), ctypes.c_int(BF16),
+                                            ctypes.c_int(n1), ctypes.c_int(d), ctypes.c_int(E * n1),
+                                            ctypes.c_int(ACTIVATIONS[activation or "none"]), ctypes.c_int(BF16),
                                             ctypes.c_int(sm_count()), _stream()))
-    hidden = glu_limited(both, inner, limit, slope, torch.bfloat16, plus)
+    hidden = both if activation is not None else glu_limited(both, inner, limit, slope, torch.bfloat16, plus)
     picked = torch.empty((max_tiles * pad, d), dtype=torch.float32, device=dev_)
     _launch(lib.ayk_gemm_tc_prefill_grouped(_ptr(picked), _ptr(hidden), _ptr(down_weight), _ptr(w_rows[1]), ctypes.c_int(max_tiles * pad),
-                                            ctypes.c_int(d), ctypes.c_int(inner), ctypes.c_int(E * d), ctypes.c_int(F32),
-                                            ctypes.c_int(sm_count()), _stream()))
+                                            ctypes.c_int(d), ctypes.c_int(inner), ctypes.c_int(E * d), ctypes.c_int(ACTIVATIONS["none"]),
+                                            ctypes.c_int(F32), ctypes.c_int(sm_count()), _stream()))
     return picked, row_of_pair
 
 

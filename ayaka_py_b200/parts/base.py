@@ -129,6 +129,12 @@ class Part:
         """``KVNeed``, ``StateNeed`` or None."""
         return None
 
+    def join_input(self, weight: torch.Tensor, bias: torch.Tensor | None) -> torch.Tensor | None:
+        """Optional, after ``bind``: another matrix [n, width] (with a bias) that reads the same rows as this part's
+        first product rides in it.  The part then leaves the extra columns, float32 [T, n], in ``ctx.carry[self]`` at
+        every forward.  Returns the matrix as a view of the stacked one; None: the part does not do this."""
+        return None
+
     def set_position(self, position: "PositionEncoding") -> None:
         """The model's position encoding, handed to every part of every layer when the
         model is built.  Parts that apply positions themselves (an attention that
@@ -147,6 +153,11 @@ class Norm(Part):
         """x: residual stream [T, d] float32 -> [T or len(rows), d] compute dtype."""
         raise NotImplementedError
 
+    def as_following(self) -> dict | None:
+        """How ``ops.stream_update`` makes this norm of the rows it has just updated (its keyword arguments);
+        None: it cannot."""
+        return None
+
 
 class Mixer(Part):
     def forward(self, h: torch.Tensor, residual: torch.Tensor, ctx, cache) -> torch.Tensor:
@@ -161,6 +172,10 @@ class FeedForward(Part):
     def forward(self, h: torch.Tensor, residual: torch.Tensor, ctx) -> torch.Tensor:
         """Returns residual + ff(h), float32 [T, d]."""
         raise NotImplementedError
+
+    def forward_rows(self, h: torch.Tensor, ctx):
+        """ff(h) for ``ops.stream_update``: float32 [T, d], or ``ops.PickedRows`` of a routed feed-forward."""
+        return self.forward(h, None, ctx)
 
 
 class PositionEncoding(Part):
@@ -192,16 +207,17 @@ class Head(Part):
 class Block:
     """Arrangement of a layer's parts: which runs on what, in which order.
 
-    ``PARTS`` names the parts the arrangement needs (a layer's spec must name
-    exactly these); each is also reachable as an attribute.  ``forward`` gets the
+    ``PARTS`` names the parts the arrangement needs, ``OPTIONAL`` those it can do without (a
+    layer's spec must name the former and no others); each is also reachable as an attribute.  ``forward`` gets the
     residual stream and, for the parts that declared a cache need, their
     ``CacheBinding`` by part name."""
 
     KIND: ClassVar[str] = ""
     PARTS: ClassVar[tuple[str, ...]] = ()
+    OPTIONAL: ClassVar[tuple[str, ...]] = ()
 
     def __init__(self, parts: dict[str, Part]):
-        missing, extra = set(self.PARTS) - set(parts), set(parts) - set(self.PARTS)
+        missing, extra = set(self.PARTS) - set(parts), set(parts) - set(self.PARTS) - set(self.OPTIONAL)
         if missing or extra:
             raise ValueError(f"arrangement {self.KIND!r} takes the parts {list(self.PARTS)}: "
                              f"missing {sorted(missing)}, not used {sorted(extra)}")
@@ -211,6 +227,14 @@ class Block:
 
     def forward(self, x: torch.Tensor, ctx, caches: dict) -> torch.Tensor:
         raise NotImplementedError
+
+    def bound(self) -> None:
+        """Called once when every part has its tensors."""
+
+    def opening_norm(self) -> "Norm | None":
+        """The norm of the stream that this arrangement starts with, when the run step before may make it (its
+        result is then in ``ctx.carry["opened"]``); None: not offered."""
+        return None
 
     def lower(self, builder, x: int, caches: dict) -> int:
         """Optional, as ``Part.lower``: the arrangement over buffers."""

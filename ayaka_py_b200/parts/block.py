@@ -2,6 +2,7 @@
 
 from __future__ import annotations
 
+from .. import ops
 from .base import Block, register_block
 
 
@@ -112,3 +113,60 @@ class DoubleNormMixerBlock(DoubleNormBlock):
 
 register_block(DoubleNormBlock.KIND, DoubleNormBlock)
 register_block(DoubleNormMixerBlock.KIND, DoubleNormMixerBlock)
+
+
+class GatedPreNormBlock(Block):
+    """A norm in front of each sublayer, a constant and a gate per channel behind it (``ResidualGate``), and a token's
+    row of a side table at the layer's end (``TokenSide``):
+    x += s1 g1(h) mixer(h) with h = norm1(x); x += s2 g2(h) ffn(h) with h = norm2(x); x += side(x, token).
+    The feed-forward (with its norm and gate) and the side input may be absent.  The gates' products ride in the
+    sublayers' first products; every update of the stream is one kernel that also makes what the next product reads
+    (``ops.stream_update``), the next layer's opening norm included."""
+
+    KIND = "gated_pre_norm"
+    PARTS = ("norm1", "mixer", "gate1")
+    OPTIONAL = ("norm2", "ffn", "gate2", "side")
+
+    def __init__(self, parts):
+        super().__init__(parts)
+        together = [name in parts for name in ("norm2", "ffn", "gate2")]
+        if any(together) and not all(together):
+            raise ValueError(f"arrangement {self.KIND!r}: norm2, ffn and gate2 come together or not at all")
+
+    def bound(self):
+        self.gate1.ride(self.mixer)
+        if "ffn" in self.parts:
+            self.gate2.ride(self.ffn)
+
+    def opening_norm(self):
+        return self.norm1
+
+    @staticmethod
+    def _update(x, y, norm, ctx, **how):
+        """The stream takes up y; returns ``norm`` of it (None: nothing), from the same kernel where that can be."""
+        post = norm.as_following() if norm is not None else None
+        h = ops.stream_update(x, y, **how, **(post or {}))
+        return norm.forward(x, ctx) if norm is not None and post is None else h
+
+    def forward(self, x, ctx, caches):
+        h = ctx.carry.pop("opened", None)
+        if h is None:
+            h = self.norm1.forward(x, ctx)
+        y, gate = self.mixer.forward(h, None, ctx, caches.get("mixer")), self.gate1
+        gates = gate.gates(self.mixer, h, ctx)
+        if "ffn" in self.parts:
+            h = self._update(x, y, self.norm2, ctx, scale=gate.scale, gate=gates)
+            y, gate = self.ffn.forward_rows(h, ctx), self.gate2
+            gates = gate.gates(self.ffn, h, ctx)
+        if "side" in self.parts:
+            copies = {"post": "copy", "out_dtype": self.side.dtype} if self.side.reads_copy(x.shape[0]) else {}
+            copy = ops.stream_update(x, y, gate.scale, gate=gates, **copies)
+            opened = self._update(x, self.side.forward(x, copy, ctx), ctx.following, ctx, scale=self.side.norm, eps=self.side.eps)
+        else:
+            opened = self._update(x, y, ctx.following, ctx, scale=gate.scale, gate=gates)
+        if opened is not None:
+            ctx.carry["opened"] = opened
+        return x
+
+
+register_block(GatedPreNormBlock.KIND, GatedPreNormBlock)

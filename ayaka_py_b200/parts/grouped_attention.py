@@ -1,6 +1,6 @@
-"""Two softmax attentions over the paged cache that share one set of kernels (``csrc/attention_grouped.cu``):
-per-head RMS norm of queries and keys with one weight for all heads, keys and values grouped separately, a
-window, no rotation.
+"""Three softmax attentions over the paged cache that share one set of kernels (``csrc/attention_grouped.cu``).
+The first two: per-head RMS norm of queries and keys with one weight for all heads, keys and values grouped
+separately, a window, no rotation.
 
 ``talking_attention``: q = W_q h + b_q, k = W_k h + b_k; the values are the projected keys as they are before
 their norm.  The score of head g is (q_g . k) scale temp_g - slope_g (i - j) with slope_g = 2^(-c (g + 1) / H);
@@ -17,7 +17,13 @@ its own run of that many positions (runs counted from position 0 of the sequence
 output is multiplied by sigmoid(W_g h)_h, one number per head, before the output projection.  The kernel sees
 2 H query heads, 2 G key heads and G value heads.
 
-Norms, scores, weights, the mix and lambda are 32-bit in both dtypes."""
+``rotary_attention``: grouped queries without norms or biases; the first ``rot.dims`` dimensions of every query and
+key head turn by the position (dimension i with i + dims/2); a window; with ``sink`` = s the softmax's denominator has
+exp(s) more (one more key, always seen, that has no value).  ``value_mix``: "first" leaves the layer's values for the
+later layers of the same step, "blend" files (1 - lambda) v + lambda v_first in the place of its own values v, lambda a
+tensor of the layer (``csrc/rotary_prepare.cu``).
+
+Norms, angles, scores, weights, the mixes and lambda are 32-bit in both dtypes."""
 
 from __future__ import annotations
 
@@ -26,7 +32,8 @@ import math
 import torch
 
 from .. import ops
-from .base import KVNeed, Mixer, TensorDecl, register_part
+from .base import KVNeed, Mixer, PartSpec, TensorDecl, make_part, register_part
+from .stacked import StackedInput
 
 
 def _padded(n: int) -> int:
@@ -160,5 +167,80 @@ class DifferentialAttention(Mixer):
         return ops.linear(o, self.out_weight, None, residual=residual, out_dtype=torch.float32, out=residual)
 
 
+class RotaryAttention(Mixer):
+    KIND = "rotary_attention"
+    FIRST_VALUES = "first_values"            # the name in ``ctx.carry``
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rot: dict | None = None,
+                 window: int | None = None, sink: float | None = None, value_mix: str | None = None,
+                 dtype=torch.float32, device="cuda"):
+        _check_heads(heads, kv_heads, dim, vdim)
+        if dim > 1024:
+            raise ValueError(f"heads of {dim} numbers: the attention kernels take keys of up to 1024")
+        if rot is not None and rot["dims"] > dim:
+            raise ValueError(f"{rot['dims']} rotated dimensions do not fit a head of {dim}")
+        if value_mix not in (None, "first", "blend"):
+            raise ValueError(f"value_mix {value_mix!r}: 'first', 'blend' or None")
+        self.width, self.heads, self.kv_heads, self.dim, self.vdim = width, heads, kv_heads, dim, vdim
+        self.scale, self.window, self.sink, self.value_mix, self.dtype = float(scale), window, sink, value_mix, dtype
+        self.rotary = None
+        if rot is not None:
+            self.rotary = make_part(PartSpec("rotary", {"dims": rot["dims"], "base": rot["base"], "layout": "halves"}), dtype, device)
+        self.stack = self.sinks = self.joined = None
+        self.lam = 0.0
+
+    def tensors(self):
+        d = self.width
+        out = {"q_weight": TensorDecl((self.heads * self.dim, d), "matrix"), "k_weight": TensorDecl((self.kv_heads * self.dim, d), "matrix"),
+               "v_weight": TensorDecl((self.kv_heads * self.vdim, d), "matrix"),
+               "out_weight": TensorDecl((d, self.heads * self.vdim), "matrix")}
+        if self.value_mix is not None:
+            out["mix"] = TensorDecl((), "vector")
+        return out
+
+    def bind(self, tensors):
+        """q | k | v become one product."""
+        super().bind(tensors)
+        self.stack = StackedInput(self.width, [[self.q_weight, self.k_weight, self.v_weight]])
+        self._take_views()
+        if self.value_mix == "blend":
+            self.lam = float(self.mix)
+        if self.sink is not None:
+            self.sinks = torch.full((self.heads,), float(self.sink), dtype=torch.float32, device=self.stack.weight.device)
+
+    def _take_views(self) -> None:
+        self.q_weight, self.k_weight, self.v_weight = self.stack.views[:3]
+
+    def join_input(self, weight, bias):
+        at = self.stack.join(weight, bias)
+        self._take_views()
+        self.joined = (at, at + weight.shape[0])
+        return self.stack.views[-1]
+
+    def cache_need(self):
+        return KVNeed(kv_heads=self.kv_heads, head_dim=self.dim, window=self.window, value_heads=self.kv_heads, value_dim=self.vdim)
+
+    def forward(self, h, residual, ctx, cache):
+        """residual + mix(h); with ``residual`` None the mixer's output alone, float32 [T, width]."""
+        kpages, vpages = ctx.cache.kv_layer(cache.group, cache.layer)
+        table = ctx.tables[cache.group]
+        H, G, D = self.heads, self.kv_heads, self.dim
+        proj = ops.linear(h, self.stack.weight, self.stack.bias, out_dtype=torch.float32)
+        first = None
+        if self.value_mix == "first":
+            ctx.carry[self.FIRST_VALUES] = proj[:, (H + G) * D:(H + G) * D + G * self.vdim]
+        elif self.value_mix == "blend":
+            first = ctx.carry[self.FIRST_VALUES]
+        if self.joined is not None:
+            ctx.carry[self] = proj[:, self.joined[0]:self.joined[1]]
+        rot = self.rotary
+        q = ops.rotary_prepare(proj, kpages, vpages, rot.freq if rot else None, rot.dims if rot else 0, ctx, table, H, cache.writes,
+                               self.dtype, first=first, mix=self.lam)
+        o = ops.grouped_attention(q, kpages, vpages, table, ctx, heads=H, key_heads=G, key_dim=D, scale=self.scale,
+                                  window=self.window, sinks=self.sinks)
+        return ops.linear(o, self.out_weight, None, residual=residual, out_dtype=torch.float32, out=residual)
+
+
+register_part(RotaryAttention.KIND, RotaryAttention)
 register_part(TalkingAttention.KIND, TalkingAttention)
 register_part(DifferentialAttention.KIND, DifferentialAttention)

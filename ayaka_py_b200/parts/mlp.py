@@ -8,6 +8,7 @@ import torch
 
 from .. import ops
 from .base import FeedForward, TensorDecl, register_part
+from .stacked import StackedInput
 
 
 class MLP(FeedForward):
@@ -67,15 +68,19 @@ class PolyNormMLP(FeedForward):
 
 class GatedMLP(FeedForward):
     """down(act(gate h) * (up h)) without biases.  gate | up is one product, stored in 32-bit; the
-    activation and the product of the halves are 32-bit, their result is stored in the compute dtype."""
+    activation and the product of the halves are 32-bit, their result is stored in the compute dtype.
+    ``activation`` "limited_glu": g sigmoid(slope g) (u + plus) with g = min(gate h, limit) and
+    u = clamp(up h, -limit, limit) instead."""
 
     KIND = "gated_mlp"
 
-    def __init__(self, width: int, inner: int, activation: str, dtype=torch.float32, device="cuda"):
-        if activation not in ops.ACTIVATIONS:
-            raise ValueError(f"unknown activation {activation!r}; known: {sorted(ops.ACTIVATIONS)}")
+    def __init__(self, width: int, inner: int, activation: str, limit: float | None = None, slope: float = 1.702, plus: float = 1.0,
+                 dtype=torch.float32, device="cuda"):
+        if activation != "limited_glu" and activation not in ops.ACTIVATIONS:
+            raise ValueError(f"unknown activation {activation!r}; known: {sorted(ops.ACTIVATIONS)} and 'limited_glu'")
         self.width, self.inner, self.activation, self.dtype = width, inner, activation, dtype
-        self.gate_weight = self.up_weight = self.down_weight = self.in_weight = None
+        self.limit, self.slope, self.plus = float("inf") if limit is None else float(limit), float(slope), float(plus)
+        self.gate_weight = self.up_weight = self.down_weight = self.stack = self.joined = None
 
     def tensors(self):
         return {"gate_weight": TensorDecl((self.inner, self.width), "matrix"),
@@ -84,13 +89,28 @@ class GatedMLP(FeedForward):
 
     def bind(self, tensors):
         super().bind(tensors)
-        self.in_weight = torch.cat([self.gate_weight, self.up_weight], dim=0).contiguous()
-        self.gate_weight, self.up_weight = self.in_weight[:self.inner], self.in_weight[self.inner:]
+        self.stack = StackedInput(self.width, [[self.gate_weight, self.up_weight]])
+        self.gate_weight, self.up_weight = self.stack.views[:2]
+
+    @property
+    def in_weight(self):
+        return self.stack.weight
+
+    def join_input(self, weight, bias):
+        at = self.stack.join(weight, bias)
+        self.gate_weight, self.up_weight = self.stack.views[:2]
+        self.joined = (at, at + weight.shape[0])
+        return self.stack.views[-1]
 
     def forward(self, h, residual, ctx):
         """residual + ff(h); with ``residual`` None the sublayer's output alone, float32."""
-        z = ops.linear(h, self.in_weight, None, out_dtype=torch.float32)
-        u = ops.gated_act(z, self.inner, self.activation, self.dtype)
+        z = ops.linear(h, self.stack.weight, self.stack.bias, out_dtype=torch.float32)
+        if self.joined is not None:
+            ctx.carry[self] = z[:, self.joined[0]:self.joined[1]]
+        if self.activation == "limited_glu":
+            u = ops.glu_limited(z, self.inner, self.limit, self.slope, self.dtype, self.plus)
+        else:
+            u = ops.gated_act(z, self.inner, self.activation, self.dtype)
         return ops.linear(u, self.down_weight, None, residual=residual, out_dtype=torch.float32, out=residual)
 
 

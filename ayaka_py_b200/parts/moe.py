@@ -13,7 +13,9 @@ equal runs of consecutive experts (a run's score: the sum of its two largest ran
 chosen at all), and weights the chosen experts by s over their sum, times ``route_scale``.  ``slope`` and
 ``plus`` set the activation g sigmoid(slope g) (u + plus); a limit of None clamps nothing (slope 1, plus 0,
 no limit: silu(gate) * up).  ``shared_gated`` False: the shared expert is added as it is;
-``shared_inner`` 0: there is none.
+``shared_inner`` 0: there is none.  ``router="softmax_groups"``: s = softmax(z) over all experts, experts ranked by s,
+a run's score its largest s, the weights the chosen s as they are, times ``route_scale``.  ``activation``: experts
+without a gate, y = W_down act(W_up h) (no shared expert then).
 
 The experts' matrices are kept stacked ([experts, 2 inner, width] with gate over up, and
 [experts, width, inner]); a step sorts its (token, choice) pairs by expert on the device and runs
@@ -28,6 +30,7 @@ import torch
 
 from .. import ops
 from .base import FeedForward, TensorDecl, register_part
+from .stacked import StackedInput
 
 
 def _padded(n: int) -> int:
@@ -41,12 +44,14 @@ class MoE(FeedForward):
     def __init__(self, width: int, experts: int, top: int, inner: int, limit: float | None, shared_inner: int,
                  shared_limit: float | None, router: str = "softmax", groups: int = 1, keep: int = 1,
                  route_scale: float = 1.0, slope: float = GATE_SLOPE, plus: float = 1.0, shared_gated: bool = True,
-                 dtype=torch.float32, device="cuda"):
+                 activation: str | None = None, dtype=torch.float32, device="cuda"):
         if not 1 <= top <= min(experts, 16):
             raise ValueError(f"top {top} of {experts} experts: the routing kernel picks 1 to 16")
-        if router not in ("softmax", "sigmoid_groups"):
-            raise ValueError(f"unknown router {router!r}; known: softmax, sigmoid_groups")
-        if router == "sigmoid_groups" and not (1 <= keep <= groups <= 32 and experts % groups == 0 and keep * (experts // groups) >= top):
+        if router not in ("softmax", "sigmoid_groups", "softmax_groups"):
+            raise ValueError(f"unknown router {router!r}; known: softmax, sigmoid_groups, softmax_groups")
+        if activation is not None and (activation not in ops.ACTIVATIONS or shared_inner):
+            raise ValueError(f"experts without a gate take one of {sorted(ops.ACTIVATIONS)} and no shared expert, got {activation!r}")
+        if router != "softmax" and not (1 <= keep <= groups <= 32 and experts % groups == 0 and keep * (experts // groups) >= top):
             raise ValueError(f"{experts} experts in {groups} groups (at most 32) of which {keep} are kept cannot give {top} choices")
         self.width, self.experts, self.top, self.inner = width, experts, top, inner
         self.limit = float("inf") if limit is None else float(limit)
@@ -54,7 +59,8 @@ class MoE(FeedForward):
         self.shared_limit = float("inf") if shared_limit is None else float(shared_limit)
         self.router, self.groups, self.keep, self.route_scale = router, int(groups), int(keep), float(route_scale)
         self.slope, self.plus, self.shared_gated = float(slope), float(plus), bool(shared_gated) and shared_inner > 0
-        self.correction = None
+        self.activation = activation
+        self.correction = self.stack = self.joined = None
         # many pairs in bfloat16, rows in whole 16-byte pieces: the experts' products run on tcgen05
         self.tensor_cores = dtype == torch.bfloat16 and width % 8 == 0 and inner % 8 == 0
 
@@ -69,22 +75,24 @@ class MoE(FeedForward):
         if self.shared_gated:
             out["shared_mix"] = TensorDecl((1, d), "matrix")
         for e in range(self.experts):
-            out[f"gate_{e}"] = TensorDecl((ff, d), "matrix")
+            if self.activation is None:
+                out[f"gate_{e}"] = TensorDecl((ff, d), "matrix")
             out[f"up_{e}"] = TensorDecl((ff, d), "matrix")
             out[f"down_{e}"] = TensorDecl((d, ff), "matrix")
         return out
 
     def bind(self, tensors):
         E, d, ff, sf = self.experts, self.width, self.inner, self.shared_inner
-        first = tensors["gate_0"]
-        self.in_weight = torch.empty((E, 2 * ff, d), dtype=first.dtype, device=first.device)
+        first, gated = tensors["up_0"], self.activation is None
+        self.in_weight = torch.empty((E, 2 * ff if gated else ff, d), dtype=first.dtype, device=first.device)
         self.down_weight = torch.empty((E, d, ff), dtype=first.dtype, device=first.device)
         for e in range(E):
-            self.in_weight[e, :ff], self.in_weight[e, ff:] = tensors[f"gate_{e}"], tensors[f"up_{e}"]
+            if gated:
+                self.in_weight[e, :ff] = tensors[f"gate_{e}"]
+            self.in_weight[e, -ff:] = tensors[f"up_{e}"]
             self.down_weight[e] = tensors[f"down_{e}"]
-        rows = _padded(max(E, 8))
-        self.router_weight = torch.zeros((rows, d), dtype=first.dtype, device=first.device)
-        self.router_weight[:E] = tensors["router_weight"]
+        self.stack = StackedInput(d, [[tensors["router_weight"]]])
+        self.router_weight = self.stack.views[0]
         if "correction" in tensors:
             self.correction = tensors["correction"]
         if sf:
@@ -94,33 +102,51 @@ class MoE(FeedForward):
                 self.shared_in[2 * sf] = tensors["shared_mix"][0]
             self.shared_down = tensors["shared_down"]
         for e in range(E):                         # per-expert views, as the loader's bookkeeping expects attributes
-            setattr(self, f"gate_{e}", self.in_weight[e, :ff])
-            setattr(self, f"up_{e}", self.in_weight[e, ff:])
+            if gated:
+                setattr(self, f"gate_{e}", self.in_weight[e, :ff])
+            setattr(self, f"up_{e}", self.in_weight[e, -ff:])
             setattr(self, f"down_{e}", self.down_weight[e])
         if sf:
             self.shared_gate, self.shared_up = self.shared_in[:sf], self.shared_in[sf:2 * sf]
         if self.shared_gated:
             self.shared_mix = self.shared_in[2 * sf:2 * sf + 1]
 
+    def join_input(self, weight, bias):
+        """Another matrix rides in the router's product."""
+        at = self.stack.join(weight, bias)
+        self.router_weight = self.stack.views[0]
+        self.joined = (at, at + weight.shape[0])
+        return self.stack.views[-1]
+
+    def _experts(self, h, ctx):
+        """The chosen experts' rows: (float32 rows, routing, row of every pair or None)."""
+        pairs = h.shape[0] * self.top
+        logits = ops.linear(h, self.stack.weight, self.stack.bias, out_dtype=torch.float32)
+        if self.joined is not None:
+            ctx.carry[self] = logits[:, self.joined[0]:self.joined[1]]
+        scored = None
+        if self.router != "softmax":
+            scored = {"correction": self.correction, "groups": self.groups, "keep": self.keep, "factor": self.route_scale}
+        if self.router == "softmax_groups":
+            scored.update(scores="softmax", group_best=1, normalize=False)
+        route = ops.moe_route(logits, self.experts, self.top, scored)
+        act = self.activation
+        glu = (self.limit, self.slope, self.plus)
+        if self.tensor_cores and pairs >= ops.MOE_TENSOR_PAIRS:
+            picked, rows = ops.moe_experts_tc(h, self.in_weight, self.down_weight, route, *glu, activation=act)
+            return picked, rows, route
+        glu = glu if act is None else None
+        if self.tensor_cores and ops.moe_gemv_takes(h, self.in_weight):
+            # a handful of pairs (a step of single tokens): every pair streams its expert's matrices on its own
+            hidden = ops.moe_gemv(h, self.in_weight, route, glu=glu, activation=act)
+            return ops.moe_gemv(hidden, self.down_weight, route, glu=None), None, route                    # [T * K, d]
+        hidden = ops.moe_gemm(h, self.in_weight, route, glu=glu, out_dtype=self.dtype, activation=act)
+        return ops.moe_gemm(hidden, self.down_weight, route, glu=None, out_dtype=torch.float32), None, route
+
     def forward(self, h, residual, ctx):
         """ff(h) (+ residual), float32 [T, width].  h: rows in the compute dtype."""
-        T, d, K = h.shape[0], self.width, self.top
-        logits = ops.linear(h, self.router_weight, None, out_dtype=torch.float32)
-        scored = None
-        if self.router == "sigmoid_groups":
-            scored = {"correction": self.correction, "groups": self.groups, "keep": self.keep, "factor": self.route_scale}
-        route = ops.moe_route(logits, self.experts, K, scored)
-        rows = None
-        glu = (self.limit, self.slope, self.plus)
-        if self.tensor_cores and T * K >= ops.MOE_TENSOR_PAIRS:
-            picked, rows = ops.moe_experts_tc(h, self.in_weight, self.down_weight, route, *glu)
-        elif self.tensor_cores and ops.moe_gemv_takes(h, self.in_weight):
-            # a handful of pairs (a step of single tokens): every pair streams its expert's matrices on its own
-            hidden = ops.moe_gemv(h, self.in_weight, route, glu=glu)
-            picked = ops.moe_gemv(hidden, self.down_weight, route, glu=None)                               # [T * K, d]
-        else:
-            hidden = ops.moe_gemm(h, self.in_weight, route, glu=glu, out_dtype=self.dtype)
-            picked = ops.moe_gemm(hidden, self.down_weight, route, glu=None, out_dtype=torch.float32)      # [T * K, d]
+        T, d = h.shape[0], self.width
+        picked, rows, route = self._experts(h, ctx)
         if self.shared_inner:
             sp = ops.linear(h, self.shared_in, None, out_dtype=torch.float32)
             sh = ops.glu_limited(sp, self.shared_inner, self.shared_limit, self.slope, self.dtype, self.plus)
@@ -132,6 +158,13 @@ class MoE(FeedForward):
             residual.add_(out)
             return residual
         return out
+
+    def forward_rows(self, h, ctx):
+        """Without a shared expert the chosen experts' rows themselves: their sum is left to the kernel that needs it."""
+        if self.shared_inner:
+            return self.forward(h, None, ctx)
+        picked, rows, route = self._experts(h, ctx)
+        return ops.PickedRows(picked, route, rows)
 
 
 register_part(MoE.KIND, MoE)

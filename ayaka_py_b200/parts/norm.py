@@ -29,6 +29,9 @@ class LayerNorm(Norm):
     def lower(self, builder, x, wanted=False):
         return builder.layernorm(x, self.weight, self.bias, self.eps, self.width, self.dtype, wanted=wanted)
 
+    def as_following(self):
+        return {"post": "layernorm", "next_weight": self.weight, "next_bias": self.bias, "next_eps": self.eps, "out_dtype": self.dtype}
+
     def add_normed(self, x, y):
         """x += norm(y), in place; x and y float32 [T, width]: a norm that closes a sublayer."""
         ops.layernorm_residual(x, y, self.weight, self.bias, self.eps)
@@ -76,6 +79,11 @@ class RMSNorm(Norm):
         if self.out_scale != 1.0:
             raise ValueError("an RMS norm with an output factor only adds to the residual stream (add_normed)")
         return ops.rmsnorm(x, self.weight, self.eps, self.dtype, rows=rows, groups=self.groups)
+
+    def as_following(self):
+        if self.groups != 1 or self.out_scale != 1.0:
+            return None
+        return {"post": "rmsnorm", "next_weight": self.weight, "next_eps": self.eps, "out_dtype": self.dtype}
 
     def add_normed(self, x, y):
         """x += out_scale * norm(y), in place; x and y float32 [T, width]."""

@@ -208,6 +208,8 @@ def load_weights(model, store: TensorStore, normalize_name=None, config=None) ->
         per_part.setdefault(id(row.part), (row.part, {}))[1][row.name] = shared[key]
     for part, tensors in per_part.values():
         part.bind(tensors)
+    for block in model.blocks:
+        block.bound()
     if str(model.device).startswith("cuda"):
         torch.cuda.synchronize()
     model.loaded = True
