@@ -19,6 +19,12 @@
 // whatever carries a decay or the state (S_0, the scores times their decay, the decayed values) enters its
 // product as two bfloat16 parts, the rounding and the remainder, so that the products see 16 bits of them; sums
 // are 32-bit and S itself stays in 32-bit registers.
+//
+// Long portions take the chunks side by side instead of one after the other, three launches: what every chunk adds
+// to the memory, sum_s lambda^(L-1-s) k_s v_s^T, in float32 scratch (decay_chunk_sum_kernel); the walk over a
+// request's chunks, which is now a sum per cell of S and leaves every chunk's S_0 in the place of what the chunk
+// added (decay_chunk_scan_kernel); and the outputs of every chunk from its S_0 (decay_chunk_out_kernel).  The
+// arithmetic is the same.
 #include <math.h>
 
 #include "common.cuh"
@@ -37,7 +43,7 @@ __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 constexpr int WWARPS = 8, WCOLS = 32, WTOK = 16;
 
 template <int DP>          // rows of S per thread, at most
-__global__ void __launch_bounds__(WWARPS * 32)
+__global__ void __launch_bounds__(WWARPS * 32, DP <= 16 ? 4 : 1)
 decay_walk_kernel(float* __restrict__ out, float* __restrict__ state, const float* __restrict__ proj, long long stride,
                   const float* __restrict__ powers, const int* __restrict__ req_q_start, const int* __restrict__ req_slot,
                   int H, int D, int DV, int settled) {
@@ -413,6 +419,328 @@ int launch_chunk(float* out, float* state, const __nv_bfloat16* qkv, long long s
   return ayk_check_launch("ayk_decay_chunk");
 }
 
+// ------------------------------------------------------- chunks side by side --
+// which chunk of which request is global chunk number c?  (chunks are numbered request by request)
+__device__ __forceinline__ bool find_chunk(const int* req_q_start, int R, int c, int& req, int& t0) {
+  for (int r = 0; r < R; ++r) {
+    const int chunks = (req_q_start[r + 1] - req_q_start[r] + DECAY_CHUNK - 1) / DECAY_CHUNK;
+    if (c < chunks) { req = r; t0 = c * DECAY_CHUNK; return true; }
+    c -= chunks;
+  }
+  return false;
+}
+
+// 64 rows of ``n`` numbers (n16 = n rounded up to 16, or the width of a slice) from ``src`` into shared rows of ld;
+// rows from L on and columns from n on are zeros.  ``vec``: 16-byte pieces, copied asynchronously.
+template <int THREADS>
+__device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, long long stride, int n, int n16, int L,
+                                           bool vec) {
+  if (vec) {
+    const int pieces = n16 / 8;
+    for (int t = threadIdx.x >> 3; t < DECAY_CHUNK; t += THREADS / 8)
+      for (int p = threadIdx.x & 7; p < pieces; p += 8) {
+        const bool live = t < L && p * 8 < n;
+        cp_async_16(dst + t * ld + p * 8, live ? src + (size_t)t * stride + p * 8 : src, live);
+      }
+  } else {
+    for (int t = threadIdx.x >> 5; t < DECAY_CHUNK; t += THREADS / 32)
+      for (int d = threadIdx.x & 31; d < n16; d += 32)
+        dst[t * ld + d] = (t < L && d < n) ? src[(size_t)t * stride + d] : __float2bfloat16_rn(0.f);
+  }
+}
+
+__host__ __device__ inline size_t decay_sum_bytes(int D, int COLS) {
+  const int LDK = ((D + 15) & ~15) + 8, LDV = COLS + 8;
+  return ((size_t)DECAY_CHUNK * LDK + (size_t)3 * DECAY_CHUNK * LDV) * sizeof(__nv_bfloat16) + (DECAY_CHUNK + 4) * sizeof(float);
+}
+
+// scratch [chunk][H][D][DV] = sum_s lambda^(L-1-s) k_s v_s^T.  Block (8 NT value columns, head, chunk), four warps.
+template <int MT, int NT>
+__global__ void __launch_bounds__(CWARPS * 32)
+decay_chunk_sum_kernel(float* __restrict__ scratch, const __nv_bfloat16* __restrict__ qkv, long long stride,
+                       const float* __restrict__ powers, const int* __restrict__ req_q_start, int R, int H, int D, int DV, int vec) {
+  constexpr int CT = DECAY_CHUNK, COLS = NT * 8, LDV = COLS + 8, THREADS = CWARPS * 32;
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int D16 = (D + 15) & ~15, LDK = D16 + 8;
+  __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);     // [CT][LDK]
+  __nv_bfloat16* Vs = Ks + CT * LDK;                                  // [CT][LDV]
+  __nv_bfloat16* Vh = Vs + CT * LDV;
+  __nv_bfloat16* Vl = Vh + CT * LDV;
+  float* pw = reinterpret_cast<float*>(Vl + CT * LDV);
+  pdl_trigger();
+  const int c0 = blockIdx.x * COLS, h = blockIdx.y;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+  int req = 0, t0 = 0;
+  if (!find_chunk(req_q_start, R, blockIdx.z, req, t0)) return;
+  const int first = req_q_start[req] + t0, L = min(CT, req_q_start[req + 1] - first);
+  for (int i = tid; i <= CT; i += THREADS) pw[i] = powers[h * (CT + 1) + i];
+  pdl_wait();
+  const __nv_bfloat16* row0 = qkv + (size_t)first * stride;
+  fetch_rows<THREADS>(Ks, LDK, row0 + H * D + h * D, stride, D, D16, L, vec);
+  fetch_rows<THREADS>(Vs, LDV, row0 + 2 * H * D + h * DV + c0, stride, DV - c0, COLS, L, vec);
+  asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  for (int i = tid; i < CT * COLS / 2; i += THREADS) {
+    const int t = i / (COLS / 2), c = (i - t * (COLS / 2)) * 2;
+    const float w = t < L ? pw[L - 1 - t] : 0.f;
+    const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(Vs + t * LDV + c);
+    uint32_t hi, lo;
+    split_bf16(w * __low2float(v), w * __high2float(v), hi, lo);
+    *reinterpret_cast<uint32_t*>(Vh + t * LDV + c) = hi;
+    *reinterpret_cast<uint32_t*>(Vl + t * LDV + c) = lo;
+  }
+  __syncthreads();
+  const int a_at = ((lane & 7) + (lane >> 4) * 8) * LDK + ((lane >> 3) & 1) * 8;
+  const int v_at = ((lane & 7) + ((lane >> 3) & 1) * 8) * LDV + (lane >> 4) * 8;
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) acc[i][j][c] = 0.f;
+#pragma unroll
+  for (int ks = 0; ks < CT / 16; ++ks) {
+    if (ks * 16 >= L) break;
+    uint32_t bh[NT / 2][4], bl[NT / 2][4];
+#pragma unroll
+    for (int np = 0; np < NT / 2; ++np) {
+      ldmatrix_x4_trans(bh[np], smem_addr(Vh + ks * 16 * LDV + np * 16 + v_at));
+      ldmatrix_x4_trans(bl[np], smem_addr(Vl + ks * 16 * LDV + np * 16 + v_at));
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i) {
+      const int tile = warp + CWARPS * i;
+      if (tile * 16 >= D16) break;
+      uint32_t af[4];
+      ldmatrix_x4_trans(af, smem_addr(Ks + ks * 16 * LDK + tile * 16 + a_at));
+#pragma unroll
+      for (int np = 0; np < NT / 2; ++np) {
+        mma_bf16(acc[i][2 * np], af, bh[np][0], bh[np][1]);
+        mma_bf16(acc[i][2 * np + 1], af, bh[np][2], bh[np][3]);
+        mma_bf16(acc[i][2 * np], af, bl[np][0], bl[np][1]);
+        mma_bf16(acc[i][2 * np + 1], af, bl[np][2], bl[np][3]);
+      }
+    }
+  }
+  float* dst = scratch + ((size_t)blockIdx.z * H + h) * D * DV;
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int row = (warp + CWARPS * i) * 16 + gid + half * 8, col = c0 + j * 8 + tig * 2;
+        if (row >= D || col >= DV) continue;
+        float* at = dst + (size_t)row * DV + col;
+        if (DV % 2 == 0) {
+          *reinterpret_cast<float2*>(at) = make_float2(acc[i][j][half * 2], acc[i][j][half * 2 + 1]);
+        } else {
+          at[0] = acc[i][j][half * 2];
+          if (col + 1 < DV) at[1] = acc[i][j][half * 2 + 1];
+        }
+      }
+}
+
+// Per four cells of S: the walk over a request's chunks; scratch gets every chunk's S_0, the state the last S.
+__global__ void __launch_bounds__(128)
+decay_chunk_scan_kernel(float* __restrict__ scratch, float* __restrict__ state, const float* __restrict__ powers,
+                        const int* __restrict__ req_q_start, const int* __restrict__ req_slot, int H, int cells) {
+  constexpr int AHEAD = 8;
+  pdl_trigger();
+  const int i = (blockIdx.x * 128 + threadIdx.x) * 4, h = blockIdx.y, r = blockIdx.z;
+  int chunk0 = 0;
+  for (int q = 0; q < r; ++q) chunk0 += (req_q_start[q + 1] - req_q_start[q] + DECAY_CHUNK - 1) / DECAY_CHUNK;
+  const int n = req_q_start[r + 1] - req_q_start[r], chunks = (n + DECAY_CHUNK - 1) / DECAY_CHUNK;
+  const float whole = powers[h * (DECAY_CHUNK + 1) + DECAY_CHUNK];
+  const float last = powers[h * (DECAY_CHUNK + 1) + (n - (chunks - 1) * DECAY_CHUNK)];
+  pdl_wait();
+  if (i >= cells) return;
+  float* S = state + ((size_t)req_slot[r] * H + h) * cells + i;
+  float4 s = *reinterpret_cast<const float4*>(S);
+  float* at = scratch + ((size_t)chunk0 * H + h) * cells + i;
+  const size_t step = (size_t)H * cells;
+  for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+    float4 add[AHEAD];
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u)
+      if (c0 + u < chunks) add[u] = *reinterpret_cast<const float4*>(at + u * step);
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      if (c0 + u >= chunks) break;
+      *reinterpret_cast<float4*>(at + u * step) = s;
+      const float w = c0 + u == chunks - 1 ? last : whole;
+      s.x = fmaf(w, s.x, add[u].x); s.y = fmaf(w, s.y, add[u].y);
+      s.z = fmaf(w, s.z, add[u].z); s.w = fmaf(w, s.w, add[u].w);
+    }
+    at += AHEAD * step;
+  }
+  *reinterpret_cast<float4*>(S) = s;
+}
+
+__host__ __device__ inline size_t decay_out_bytes(int D, int COLS) {
+  const int D16 = (D + 15) & ~15, LDK = D16 + 8, LDV = COLS + 8;
+  return ((size_t)2 * DECAY_CHUNK * LDK + (size_t)DECAY_CHUNK * LDV + (size_t)2 * D16 * LDV) * sizeof(__nv_bfloat16) +
+         (DECAY_CHUNK + 4) * sizeof(float);
+}
+
+// The outputs of one chunk from its S_0 (scratch).  Block (8 NT value columns, head, chunk), four warps of 16 tokens.
+template <int NT>
+__global__ void __launch_bounds__(CWARPS * 32)
+decay_chunk_out_kernel(float* __restrict__ out, const float* __restrict__ scratch, const __nv_bfloat16* __restrict__ qkv,
+                       long long stride, const float* __restrict__ powers, const int* __restrict__ req_q_start, int R, int H, int D,
+                       int DV, int vec) {
+  constexpr int CT = DECAY_CHUNK, COLS = NT * 8, LDV = COLS + 8, THREADS = CWARPS * 32;
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int D16 = (D + 15) & ~15, LDK = D16 + 8;
+  __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);     // [CT][LDK]
+  __nv_bfloat16* Ks = Qs + CT * LDK;                                  // [CT][LDK]
+  __nv_bfloat16* Vs = Ks + CT * LDK;                                  // [CT][LDV]
+  __nv_bfloat16* Sh = Vs + CT * LDV;                                  // [D16][LDV]
+  __nv_bfloat16* Sl = Sh + D16 * LDV;
+  float* pw = reinterpret_cast<float*>(Sl + D16 * LDV);
+  pdl_trigger();
+  const int c0 = blockIdx.x * COLS, h = blockIdx.y;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+  int req = 0, t0 = 0;
+  if (!find_chunk(req_q_start, R, blockIdx.z, req, t0)) return;
+  const int first = req_q_start[req] + t0, L = min(CT, req_q_start[req + 1] - first);
+  for (int i = tid; i <= CT; i += THREADS) pw[i] = powers[h * (CT + 1) + i];
+  pdl_wait();
+  const __nv_bfloat16* row0 = qkv + (size_t)first * stride;
+  fetch_rows<THREADS>(Qs, LDK, row0 + h * D, stride, D, D16, L, vec);
+  fetch_rows<THREADS>(Ks, LDK, row0 + H * D + h * D, stride, D, D16, L, vec);
+  fetch_rows<THREADS>(Vs, LDV, row0 + 2 * H * D + h * DV + c0, stride, DV - c0, COLS, L, vec);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const float* S = scratch + ((size_t)blockIdx.z * H + h) * D * DV;
+#pragma unroll 4
+  for (int i = tid; i < D16 * (COLS / 4); i += THREADS) {
+    const int d = i / (COLS / 4), c = (i - d * (COLS / 4)) * 4;
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (d < D) {
+      if (DV % 4 == 0) {
+        if (c0 + c < DV) {
+          const float4 f = *reinterpret_cast<const float4*>(S + (size_t)d * DV + c0 + c);
+          v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (c0 + c + e < DV) v[e] = S[(size_t)d * DV + c0 + c + e];
+      }
+    }
+    uint2 hi, lo;
+    split_bf16(v[0], v[1], hi.x, lo.x);
+    split_bf16(v[2], v[3], hi.y, lo.y);
+    *reinterpret_cast<uint2*>(Sh + d * LDV + c) = hi;
+    *reinterpret_cast<uint2*>(Sl + d * LDV + c) = lo;
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  const int m0 = warp * 16;
+  if (m0 >= L) return;
+  float o[NT][4], sc[CT / 8][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[j][c] = 0.f;
+#pragma unroll
+  for (int j = 0; j < CT / 8; ++j)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) sc[j][c] = 0.f;
+  const uint32_t q_addr = smem_addr(Qs + (m0 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDK + (lane >> 4) * 8);
+  const uint32_t k_addr = smem_addr(Ks + ((lane >> 4) * 8 + (lane & 7)) * LDK + ((lane >> 3) & 1) * 8);
+  const int s_at = ((lane & 7) + ((lane >> 3) & 1) * 8) * LDV + (lane >> 4) * 8;
+  for (int ks = 0; ks < D16 / 16; ++ks) {
+    uint32_t qf[4];
+    ldmatrix_x4(qf, q_addr + ks * 32);
+#pragma unroll
+    for (int np = 0; np < NT / 2; ++np) {
+      uint32_t bh[4], bl[4];
+      ldmatrix_x4_trans(bh, smem_addr(Sh + s_at + ks * 16 * LDV + np * 16));
+      ldmatrix_x4_trans(bl, smem_addr(Sl + s_at + ks * 16 * LDV + np * 16));
+      mma_bf16(o[2 * np], qf, bh[0], bh[1]);
+      mma_bf16(o[2 * np + 1], qf, bh[2], bh[3]);
+      mma_bf16(o[2 * np], qf, bl[0], bl[1]);
+      mma_bf16(o[2 * np + 1], qf, bl[2], bl[3]);
+    }
+#pragma unroll
+    for (int kt = 0; kt < CT / 16; ++kt) {
+      if (kt > warp) break;
+      uint32_t bk[4];
+      ldmatrix_x4(bk, k_addr + (uint32_t)(kt * 16 * LDK + ks * 16) * 2u);
+      mma_bf16(sc[2 * kt], qf, bk[0], bk[1]);
+      mma_bf16(sc[2 * kt + 1], qf, bk[2], bk[3]);
+    }
+  }
+  const float w0 = pw[m0 + gid + 1], w1 = pw[m0 + gid + 9];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) {
+    o[j][0] *= w0; o[j][1] *= w0;
+    o[j][2] *= w1; o[j][3] *= w1;
+  }
+#pragma unroll
+  for (int kt = 0; kt < CT / 16; ++kt) {
+    if (kt > warp) break;
+    uint32_t ah[4], al[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int nt = 2 * kt + (i >> 1), half = i & 1;
+      const int t = m0 + gid + half * 8, s = nt * 8 + tig * 2;
+      const float a0 = s <= t ? sc[nt][half * 2] * pw[t - s] : 0.f;
+      const float a1 = s + 1 <= t ? sc[nt][half * 2 + 1] * pw[t - s - 1] : 0.f;
+      split_bf16(a0, a1, ah[i], al[i]);
+    }
+#pragma unroll
+    for (int np = 0; np < NT / 2; ++np) {
+      uint32_t bv[4];
+      ldmatrix_x4_trans(bv, smem_addr(Vs + s_at + kt * 16 * LDV + np * 16));
+      mma_bf16(o[2 * np], ah, bv[0], bv[1]);
+      mma_bf16(o[2 * np + 1], ah, bv[2], bv[3]);
+      mma_bf16(o[2 * np], al, bv[0], bv[1]);
+      mma_bf16(o[2 * np + 1], al, bv[2], bv[3]);
+    }
+  }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int t = m0 + gid + half * 8;
+    if (t >= L) continue;
+    float* dst = out + (size_t)(first + t) * ((size_t)H * DV) + h * DV;
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int col = c0 + j * 8 + tig * 2;
+      if (DV % 2 == 0) {
+        if (col < DV) *reinterpret_cast<float2*>(dst + col) = make_float2(o[j][half * 2], o[j][half * 2 + 1]);
+      } else {
+        if (col < DV) dst[col] = o[j][half * 2];
+        if (col + 1 < DV) dst[col + 1] = o[j][half * 2 + 1];
+      }
+    }
+  }
+}
+
+template <int MT, int NT>
+int launch_side_by_side(float* out, float* state, float* scratch, const __nv_bfloat16* qkv, long long stride, const float* powers,
+                        const int* req_q_start, const int* req_slot, int R, int chunks, int H, int D, int DV, int vec,
+                        cudaStream_t stream) {
+  const size_t sum_smem = decay_sum_bytes(D, NT * 8), out_smem = decay_out_bytes(D, NT * 8);
+  static AykPerDevice configured;
+  if (!configured.here()) {
+    cudaError_t err = cudaFuncSetAttribute(decay_chunk_sum_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (err == cudaSuccess) err = cudaFuncSetAttribute(decay_chunk_out_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (err != cudaSuccess) return ayk_fail("ayk_decay_chunks: shared memory: %s", cudaGetErrorString(err));
+    configured.here() = true;
+  }
+  const int slices = (DV + NT * 8 - 1) / (NT * 8), cells = D * DV;
+  ayk_launch(decay_chunk_sum_kernel<MT, NT>, dim3(slices, H, chunks), dim3(CWARPS * 32), sum_smem, stream, scratch, qkv, stride, powers,
+             req_q_start, R, H, D, DV, vec);
+  ayk_launch(decay_chunk_scan_kernel, dim3((cells / 4 + 127) / 128, H, R), dim3(128), 0, stream, scratch, state, powers, req_q_start,
+             req_slot, H, cells);
+  ayk_launch(decay_chunk_out_kernel<NT>, dim3(slices, H, chunks), dim3(CWARPS * 32), out_smem, stream, out, (const float*)scratch, qkv,
+             stride, powers, req_q_start, R, H, D, DV, vec);
+  return ayk_check_launch("ayk_decay_chunks");
+}
+
 // ------------------------------------------------------------------ finish --
 // out[t, :] = raw[t, :] / rms(raw[t, :]) * w * sigmoid(gate[t, :]) over a row of n numbers (all heads together).
 template <typename C, int VEC>
@@ -511,6 +839,34 @@ AYK_EXPORT int ayk_decay_chunk(float* out, float* state, const void* qkv, long l
   if (mt <= 2) AYK_DC(2, 4);
   AYK_DC(4, 4);
 #undef AYK_DC
+}
+
+// Whether the form that takes a portion's chunks side by side takes these heads.
+AYK_EXPORT int ayk_decay_chunks_takes(int D, int DV) {
+  return ayk_decay_chunk_takes(D) && D * DV % 4 == 0 && decay_out_bytes(D, 64) <= 227 * 1024;
+}
+
+// The same with all chunks of the R requests side by side (three launches).  chunks: at least as many as the requests'
+// portions have (surplus blocks leave); every request brings at least one row.  scratch: float32 [chunks][H][D][DV].
+AYK_EXPORT int ayk_decay_chunks(float* out, float* state, float* scratch, const void* qkv, long long stride, const float* powers,
+                                const int* req_q_start, const int* req_slot, int R, int chunks, int H, int D, int DV,
+                                cudaStream_t stream) {
+  if (R == 0 || chunks == 0) return 0;
+  AYK_REQUIRE(ayk_decay_chunks_takes(D, DV), "ayk_decay_chunks: heads of %d x %d", D, DV);
+  AYK_REQUIRE(H <= 65535 && R <= 65535 && chunks <= 65535, "ayk_decay_chunks: %d heads, %d requests, %d chunks", H, R, chunks);
+  const int vec = D % 8 == 0 && DV % 8 == 0 && stride % 8 == 0 && ((uintptr_t)qkv & 15) == 0;
+  const __nv_bfloat16* rows = (const __nv_bfloat16*)qkv;
+  const int mt = ((D + 15) / 16 + CWARPS - 1) / CWARPS;
+#define AYK_DS(M, N) return launch_side_by_side<M, N>(out, state, scratch, rows, stride, powers, req_q_start, req_slot, R, chunks, H, D, DV, vec, stream)
+  if (DV <= 32) {
+    if (mt <= 1) AYK_DS(1, 4);
+    if (mt <= 2) AYK_DS(2, 4);
+    AYK_DS(4, 4);
+  }
+  if (mt <= 1) AYK_DS(1, 8);
+  if (mt <= 2) AYK_DS(2, 8);
+  AYK_DS(4, 8);
+#undef AYK_DS
 }
 
 // out[t, :] = raw[t, :] / rms(raw[t, :]) * w * sigmoid(gate[t, :]), rows of n numbers; gate: float32 rows of gate_stride.

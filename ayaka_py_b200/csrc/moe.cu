@@ -547,6 +547,46 @@ glu_limited_kernel(O* __restrict__ out, const I* __restrict__ in, long long stri
     out[(size_t)blockIdx.x * n + c] = from_float<O>(glu_limited(to_float<I>(row[c]), to_float<I>(row[n + c]), limit, slope, plus));
 }
 
+// The same from 32-bit or bfloat16 rows, four columns to a thread; grid (rows, column chunks).  bfloat16 results take the
+// sigmoid from the fast exponential (a few ulp in 32-bit before the rounding).
+__device__ __forceinline__ void load_four(const float* p, float (&v)[4]) {
+  const float4 f = *reinterpret_cast<const float4*>(p);
+  v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void load_four(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+  v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+
+template <typename I, typename O>
+__global__ void __launch_bounds__(256)
+glu_limited_vec_kernel(O* __restrict__ out, const I* __restrict__ in, long long stride, int n, float limit, float slope, float plus) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
+  if (c >= n) return;
+  const I* row = in + (size_t)blockIdx.x * stride;
+  float g[4], u[4];
+  load_four(row + c, g);
+  load_four(row + n + c, u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float a = fminf(g[i], limit), b = fminf(fmaxf(u[i], -limit), limit) + plus;
+    g[i] = sizeof(O) == 2 ? __fdividef(a, 1.0f + fast_exp2(-1.4426950408889634f * slope * a)) * b : a * sigmoidf(slope * a) * b;
+  }
+  O* dst = out + (size_t)blockIdx.x * n + c;
+  if (sizeof(O) == 2) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(g[0], g[1]), hi = __floats2bfloat162_rn(g[2], g[3]);
+    uint2 packed;
+    packed.x = *reinterpret_cast<uint32_t*>(&lo);
+    packed.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = packed;
+  } else {
+    *reinterpret_cast<float4*>(dst) = make_float4(g[0], g[1], g[2], g[3]);
+  }
+}
+
 // shared[t, :] = sum_k weights[t, k] * picked[row of pair t * top + k, :] + sigmoid(mix[t]) * shared[t, :], the
 // chosen experts in the order of their choice; row_of_pair null: the pair's own number.
 __global__ void __launch_bounds__(256)
@@ -570,14 +610,15 @@ moe_combine_kernel(float* __restrict__ shared, const float* __restrict__ picked,
 
 AYK_EXPORT int ayk_moe_tile_rows() { return TILE_ROWS; }
 
-// ids, weights [T, top]; sorted [T * top]; tiles [1 + 3 * (T * top / TILE_ROWS + E)].  Two launches.
+// ids, weights [T, top]; sorted [T * top]; tiles [1 + 3 * (T * top / TILE_ROWS + E)].  Two launches; with sorted null
+// only the routing (the plan is for the products over sorted rows).
 AYK_EXPORT int ayk_moe_route(int* ids, float* weights, int* sorted, int* tiles, const float* logits, long long stride,
                              int T, int E, int top, cudaStream_t stream) {
   if (T == 0) return 0;
   AYK_REQUIRE(top >= 1 && top <= MAX_TOP && top <= E, "ayk_moe_route: top %d of %d experts (at most %d)", top, E, MAX_TOP);
   AYK_REQUIRE(E <= 4096, "ayk_moe_route: %d experts (at most 4096)", E);
   ayk_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, ids, weights, logits, stride, T, E, top);
-  ayk_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, sorted, tiles, (const int*)ids,
+  if (sorted) ayk_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, sorted, tiles, (const int*)ids,
              T * top, E);
   return ayk_check_launch("ayk_moe_route");
 }
@@ -596,7 +637,7 @@ AYK_EXPORT int ayk_moe_route_scored(int* ids, float* weights, int* sorted, int* 
   AYK_REQUIRE(group_best == 1 || group_best == 2, "ayk_moe_route_scored: a group's score is its best or its two best");
   ayk_launch(softmax ? moe_route_scored_kernel<true> : moe_route_scored_kernel<false>, dim3((T + 3) / 4), dim3(128), 0, stream, ids,
              weights, logits, stride, correction, T, E, top, groups, keep, group_best, normalize, factor);
-  ayk_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, sorted, tiles, (const int*)ids,
+  if (sorted) ayk_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, sorted, tiles, (const int*)ids,
              T * top, E);
   return ayk_check_launch("ayk_moe_route_scored");
 }
@@ -640,6 +681,16 @@ AYK_EXPORT int ayk_moe_gemm(void* out, const void* a, long long a_stride, const 
 AYK_EXPORT int ayk_glu_limited(void* out, const void* in, long long stride, int T, int n, float limit, float slope, float plus,
                                int in_dtype, int out_dtype, cudaStream_t stream) {
   if (T == 0 || n == 0) return 0;
+  if (n % 4 == 0 && stride % 4 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0 && (n + 1023) / 1024 <= 65535) {
+    const dim3 grid(T, (n + 1023) / 1024);
+#define AYK_GLU(I, O) ayk_launch(glu_limited_vec_kernel<I, O>, grid, dim3(256), 0, stream, (O*)out, (const I*)in, stride, n, limit, slope, plus)
+    if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_F32) AYK_GLU(float, float);
+    else if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_BF16) AYK_GLU(float, __nv_bfloat16);
+    else if (in_dtype == AYK_DTYPE_BF16 && out_dtype == AYK_DTYPE_BF16) AYK_GLU(__nv_bfloat16, __nv_bfloat16);
+    else return ayk_fail("ayk_glu_limited: dtypes %d -> %d", in_dtype, out_dtype);
+#undef AYK_GLU
+    return ayk_check_launch("ayk_glu_limited");
+  }
   if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_F32)
     ayk_launch(glu_limited_kernel<float, float>, dim3(T), dim3(256), 0, stream, (float*)out, (const float*)in, stride, n, limit, slope, plus);
   else if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_BF16)

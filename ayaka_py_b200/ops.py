@@ -924,13 +924,18 @@ def decay_chunk_takes(dim: int) -> bool:
     return bool(library().ayk_decay_chunk_takes(ctypes.c_int(dim)))
 
 
+DECAY_SIDE_BY_SIDE = 3    # chunks of the longest portion from which a step's portions take their chunks side by side
+
+
 def decay_recurrence(rows: torch.Tensor, state: torch.Tensor, powers: torch.Tensor, ctx, heads: int, dim: int, vdim: int,
-                     slice_cols: int = 0) -> torch.Tensor:
+                     slice_cols: int = 0, side_by_side: bool | None = None) -> torch.Tensor:
     """S <- lambda_h S + k v^T, o = S^T q per head over the step's rows, request by request, from and into ``state``
     [slots, heads, dim, vdim] float32; returns o [T, heads * vdim] float32.  ``powers`` float32 [heads, 65]:
-    lambda_h^n.  float32 ``rows`` [q | k | v | ...] before their SiLU: token by token; bfloat16 rows
-    [silu q | silu k | silu v]: 64 tokens at a time on the tensor cores (``slice_cols``: value columns per block, 16 or
-    32; 0: chosen by the grid)."""
+    lambda_h^n.  float32 ``rows`` [q | k | v | ...] before their SiLU: token by token.  bfloat16 rows
+    [silu q | silu k | silu v]: 64 tokens at a time on the tensor cores, a request's chunks one after the other
+    (``slice_cols``: value columns per block, 16 or 32; 0: chosen by the grid), or, for long portions, side by side
+    (``side_by_side``: all portions of the step so, or none; default: from three chunks on; the single-token requests,
+    which are the step's first rows, go the other way)."""
     lib = _ready()
     _f32(state, "state"); _f32(powers, "powers")
     T = rows.shape[0]
@@ -938,15 +943,30 @@ def decay_recurrence(rows: torch.Tensor, state: torch.Tensor, powers: torch.Tens
             or powers.shape != (heads, DECAY_CHUNK + 1)):
         raise KernelError("decay_recurrence: rows, state or powers do not fit")
     out = torch.empty((T, heads * vdim), dtype=torch.float32, device=rows.device)
-    common = (_ptr(out), _ptr(state), _ptr(rows), ctypes.c_longlong(rows.stride(0)), _ptr(powers), _ptr(ctx.req_q_start),
-              _ptr(ctx.req_slot), ctypes.c_int(ctx.num_requests), ctypes.c_int(heads), ctypes.c_int(dim), ctypes.c_int(vdim))
+    head = (_ptr(out), _ptr(state))
+    data = (_ptr(rows), ctypes.c_longlong(rows.stride(0)), _ptr(powers))
+    sizes = (ctypes.c_int(heads), ctypes.c_int(dim), ctypes.c_int(vdim))
     settled = ctypes.c_int(1 if getattr(ctx, "earlier_rows_settled", False) else 0)
-    if rows.dtype == torch.bfloat16:
-        _launch(lib.ayk_decay_chunk(*common, ctypes.c_int(slice_cols), settled, _stream()))
-    elif rows.dtype == torch.float32:
-        _launch(lib.ayk_decay_walk(*common, settled, _stream()))
-    else:
+    R = ctx.num_requests
+    if rows.dtype == torch.float32:
+        _launch(lib.ayk_decay_walk(*head, *data, _ptr(ctx.req_q_start), _ptr(ctx.req_slot), ctypes.c_int(R), *sizes, settled, _stream()))
+        return out
+    if rows.dtype != torch.bfloat16:
         raise KernelError(f"decay_recurrence: rows of {rows.dtype}")
+    takes = bool(lib.ayk_decay_chunks_takes(ctypes.c_int(dim), ctypes.c_int(vdim)))
+    if side_by_side is None:
+        side_by_side = takes and ctx.max_q_len > (DECAY_SIDE_BY_SIDE - 1) * DECAY_CHUNK
+    singles = min(ctx.num_single, R) if side_by_side else R
+    if singles:
+        _launch(lib.ayk_decay_chunk(*head, *data, _ptr(ctx.req_q_start), _ptr(ctx.req_slot), ctypes.c_int(singles), *sizes,
+                                    ctypes.c_int(slice_cols), settled, _stream()))
+    if singles < R:
+        chunks = (T - singles) // DECAY_CHUNK + (R - singles)
+        scratch = torch.empty((chunks * heads * dim * vdim,), dtype=torch.float32, device=rows.device)
+        _launch(lib.ayk_decay_chunks(*head, _ptr(scratch), *data, _ptr(ctx.req_q_start[singles:]), _ptr(ctx.req_slot[singles:]),
+                                     ctypes.c_int(R - singles), ctypes.c_int(chunks), *sizes, _stream()))
+        global launches
+        launches += 2
     return out
 
 
@@ -1045,14 +1065,14 @@ class MoeRoute:
         self.ids, self.weights, self.sorted, self.tiles, self.max_tiles, self.top = ids, weights, sorted_pairs, tiles, max_tiles, top
 
 
-def moe_route(logits: torch.Tensor, experts: int, top: int, scored: dict | None = None) -> MoeRoute:
+def moe_route(logits: torch.Tensor, experts: int, top: int, scored: dict | None = None, plan: bool = True) -> MoeRoute:
     """The ``top`` largest of each row's first ``experts`` float32 logits, weighted by the softmax over
     the chosen ones, and the plan of the grouped products.  ``scored`` = {correction, groups, keep, factor, scores,
     group_best, normalize}: routing by scores s of all experts instead, sigmoid (the default) or ``scores`` "softmax";
     experts are ranked by s + correction (float32 [experts] or None) among the experts of the ``keep`` best of
     ``groups`` equal runs of consecutive experts (a run's score: the sum of its two largest ranking scores, or with
     ``group_best`` 1 the largest); the weights are the chosen s over their sum (``normalize`` False: as they are),
-    times ``factor``."""
+    times ``factor``.  ``plan`` False: the routing alone (``moe_gemv`` and ``moe_experts_tc`` need no plan)."""
     lib = _ready()
     if logits.dtype != torch.float32 or logits.stride(1) != 1 or logits.shape[1] < experts:
         raise KernelError("moe_route: logits must be float32 rows of at least ``experts`` columns")
@@ -1061,8 +1081,8 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, scored: dict | None 
     max_tiles = (T * top) // rows + experts
     ids = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    sorted_pairs = torch.empty((T * top,), dtype=torch.int32, device=logits.device)
-    tiles = torch.empty((1 + 3 * max_tiles,), dtype=torch.int32, device=logits.device)
+    sorted_pairs = torch.empty((T * top,), dtype=torch.int32, device=logits.device) if plan else None
+    tiles = torch.empty((1 + 3 * max_tiles,), dtype=torch.int32, device=logits.device) if plan else None
     if scored is not None:
         correction = scored.get("correction")
         if correction is not None and _f32(correction, "correction").numel() != experts:
@@ -1078,7 +1098,7 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, scored: dict | None 
         _launch(lib.ayk_moe_route(_ptr(ids), _ptr(weights), _ptr(sorted_pairs), _ptr(tiles), _ptr(logits),
                                   ctypes.c_longlong(logits.stride(0)), ctypes.c_int(T), ctypes.c_int(experts), ctypes.c_int(top), _stream()))
     global launches
-    launches += 1
+    launches += 1 if plan else 0
     return MoeRoute(ids, weights, sorted_pairs, tiles, max_tiles, top)
 
 
@@ -1102,6 +1122,8 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | Non
     E, n_w, K = w.shape
     if a.dtype != w.dtype or a.shape[1] != K or a.stride(1) != 1 or not w.is_contiguous() or (glu is not None and activation is not None):
         raise KernelError("moe_gemm: operands do not fit")
+    if route.sorted is None:
+        raise KernelError("moe_gemm: the routing was made without a plan")
     pairs = route.sorted.numel()
     N = n_w // 2 if glu is not None else n_w
     first = glu is not None or activation is not None

@@ -129,14 +129,16 @@ class MoE(FeedForward):
             scored = {"correction": self.correction, "groups": self.groups, "keep": self.keep, "factor": self.route_scale}
         if self.router == "softmax_groups":
             scored.update(scores="softmax", group_best=1, normalize=False)
-        route = ops.moe_route(logits, self.experts, self.top, scored)
+        many = self.tensor_cores and pairs >= ops.MOE_TENSOR_PAIRS
+        few = not many and self.tensor_cores and ops.moe_gemv_takes(h, self.in_weight)
+        route = ops.moe_route(logits, self.experts, self.top, scored, plan=not many and not few)
         act = self.activation
         glu = (self.limit, self.slope, self.plus)
-        if self.tensor_cores and pairs >= ops.MOE_TENSOR_PAIRS:
+        if many:
             picked, rows = ops.moe_experts_tc(h, self.in_weight, self.down_weight, route, *glu, activation=act)
             return picked, rows, route
         glu = glu if act is None else None
-        if self.tensor_cores and ops.moe_gemv_takes(h, self.in_weight):
+        if few:
             # a handful of pairs (a step of single tokens): every pair streams its expert's matrices on its own
             hidden = ops.moe_gemv(h, self.in_weight, route, glu=glu, activation=act)
             return ops.moe_gemv(hidden, self.down_weight, route, glu=None), None, route                    # [T * K, d]

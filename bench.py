@@ -42,7 +42,9 @@ chunked differential attention, mLSTM, latent attention and group-routed experts
 same way).  ``--only vedadra`` does the same for
 the Vedadra design (talking attention and differential attention with windows, norms in groups around
 every sublayer, gated feed-forward, layers that run twice) beside GPT-2, the closest model, at equal
-width, layer runs and feed-forward weights.
+width, layer runs and feed-forward weights.  ``--only murutar``: the Murutar design (lightning recurrence, windowed
+rotary attention with a sink, gated residual branches, a side table per token, squared-ReLU experts) beside
+Tesozen, the closest model.
 """
 
 from __future__ import annotations
@@ -1372,6 +1374,286 @@ def run_tesozen(width: int, layers: int, batch: int, steps: int, warmup: int, pk
     return result
 
 
+def murutar_document(width: int, layers: int, vocab: int = 32000) -> dict:
+    """A Murutar model of real-layer sizes: heads of 128 (four query heads to a key/value head, windows of 512, half of
+    a head's dimensions turning), a lightning recurrence with a 128 x 128 memory per head, 16 experts in 4 groups of
+    which 2 experts of 2 groups run, their inner widths adding up to 2.75 x the width per token, one dense
+    feed-forward of that width, and width / 16 columns of the side table per layer."""
+    heads = width // 128
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}}, "expert": {"ff": width * 11 // 8}}
+    att = {"type": "attention",
+           "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+                     "mask": {"size": 512}, "rot": {"base": 500000.0, "dims": 64}}}
+    rec = {"type": "lightning", "mlp": moe,
+           "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(1 + 7.0 * h / heads) for h in range(heads)]}}
+    four = (rec, dict(att, mlp=moe), rec, dict(att, mlp={"kind": "dense", "ff": width * 11 // 4, "limit": 7.0}))
+    return {"architecture": "Murutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": float(width) ** 0.5},
+            "token_side": {"dim": width // 16}, "logit_softcap": 30.0, "layers": [four[i % 4] for i in range(layers)]}
+
+
+def run_murutar(width: int, layers: int, batch: int, steps: int, warmup: int, pk: dict) -> dict:
+    """Murutar beside Tesozen, the closest model (a matrix memory per head, softmax attention near the query, layer
+    norms, group-routed squared-ReLU or gated experts), at equal width, depth and active inner width (bfloat16, random
+    weights): prefill of 2 x 1,024 tokens in one step, decode of ``batch`` requests after 512-token prompts through the
+    engine (CUDA graphs), and the design's kernels one by one beside the like kernels of Tesozen at equal sizes, timed as
+    in ``run_rakalix``."""
+    import numpy as np
+    import torch
+
+    from ayaka_py_b200 import EngineConfig, Request, SamplingParams, StopCriteria, ops
+    from ayaka_py_b200.config.model import MurutarConfig, TesozenConfig
+    from ayaka_py_b200.engine.engine import Engine
+    from ayaka_py_b200.engine.loading import random_model
+    from ayaka_py_b200.engine.step import StepEntry
+
+    vocab, heads = 32000, width // 128
+    configs = {"murutar": MurutarConfig.from_dict(murutar_document(width, layers, vocab)),
+               "tesozen": TesozenConfig.from_dict(tesozen_document(width, layers, vocab))}
+    flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
+    rs = np.random.RandomState(3)
+
+    def timed(fn, reps=9):
+        for _ in range(2):
+            fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        out = []
+        for _ in range(reps):
+            flush.fill_(1.0)
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            graph.replay()
+            b.record()
+            torch.cuda.synchronize()
+            out.append(a.elapsed_time(b))
+        return sorted(out)[len(out) // 2]
+
+    result = {"width": width, "layers": layers, "batch": batch}
+    kernels = []
+
+    def kernel(name, model, ms, gbytes=None, gflop=None, like=None):
+        row = {"kernel": name, "model": model, "us": round(ms * 1e3, 1)}
+        if gbytes is not None:
+            row.update(gb_s=round(gbytes / (ms / 1e3), 1), frac=round(gbytes / (ms / 1e3) / pk["hbm_gbs"], 4), bound="hbm")
+        if gflop is not None:
+            row.update(tflops=round(gflop / ms, 2), frac=round(gflop / ms / pk["bf16_tflops"], 4), bound="bf16")
+        if like:
+            row["like"] = like
+        kernels.append(row)
+
+    for name, config in configs.items():
+        model = random_model(config, 1, "bfloat16", "cuda", generate_on_device=True)
+        engine = Engine(model, EngineConfig(dtype="bfloat16", kv_pages=batch * 64 + 130, page_size=16, max_requests=max(batch, 2),
+                                            batch_tokens=2048, prefill_chunk=2048, max_model_len=1024, decode_graph=True),
+                        eos_token_id=None)
+        cache, runner = engine.cache, engine.runner
+
+        def prefill_step():
+            slots = [cache.open(f"p{i}") for i in range(2)]
+            entries = [StepEntry(sl, 0, rs.randint(0, vocab, 1024).tolist(), [1023]) for sl in slots]
+            res = cache.reserve([(e.slot, 0, 1024) for e in entries])
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            a.record()
+            runner.run(entries)
+            b.record()
+            torch.cuda.synchronize()
+            cache.commit(res)
+            for sl in slots:
+                cache.close(sl)
+            return a.elapsed_time(b)
+        times = [prefill_step() for _ in range(7)][2:]
+        prefill_ms = sorted(times)[2]
+
+        total_new = 2 * warmup + steps + 8
+        for i in range(batch):
+            engine.submit(Request(f"d{i}", rs.randint(0, vocab, PROMPT_LEN).tolist(), SamplingParams(temperature=0.0),
+                                  StopCriteria(max_tokens=total_new, ignore_eos=True)))
+        while any(st.computed < st.prompt_len for st in engine.scheduler.states.values()):
+            engine.step()
+        for _ in range(warmup):
+            engine.step()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        a.record()
+        for _ in range(steps):
+            engine.step()
+        b.record()
+        torch.cuda.synchronize()
+        wall = time.perf_counter() - t0
+        decode_ms = a.elapsed_time(b) / steps
+        result[name] = {"prefill_tok_s": round(2048 / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
+                        "decode_tok_s": round(batch / (decode_ms / 1e3), 1), "decode_ms_per_step": round(decode_ms, 4),
+                        "decode_e2e_tok_s": round(batch * steps / wall, 1), "weight_gb": round(model.weight_bytes() / 1e9, 3),
+                        "kv_bytes_per_token": cache.bytes_per_token()}
+        for rid in list(engine.scheduler.states):
+            engine.abort(rid)
+        engine.finished.clear()
+
+        # ---- the kernels alone, on the shapes of the two steps above
+        d, T = width, 2048
+        bf, f32 = torch.bfloat16, torch.float32
+        x = torch.randn(T, d, device="cuda")
+        ctx_len = PROMPT_LEN + 64
+
+        def open_step(lengths, starts=None):
+            slots = [cache.open(f"k{i}") for i in range(len(lengths))]
+            if starts:
+                res = cache.reserve([(sl, 0, st) for sl, st in zip(slots, starts)])
+                cache.commit(res)
+            res = cache.reserve([(sl, int(cache.length[sl]), n) for sl, n in zip(slots, lengths)])
+            ctx = runner.prepare([StepEntry(sl, int(cache.length[sl]), [0] * n, []) for sl, n in zip(slots, lengths)])
+            return ctx, res, slots
+
+        for label, lengths, starts in (("prefill", [1024, 1024], None), ("decode", [1] * batch, [ctx_len] * batch)):
+            ctx, res, slots = open_step(lengths, starts)
+            rows = ctx.num_rows
+            xr = x[:rows].contiguous()
+            h = xr.to(bf)
+            y = torch.randn(rows, d, device="cuda")
+            D = 128
+            rec, att = model.blocks[0], model.blocks[1]
+            bind = {"rec": model.bindings[0]["mixer"], "att": model.bindings[1]["mixer"]}
+            st = cache.state_layer(bind["rec"].group, bind["rec"].layer)
+            kp, vp = cache.kv_layer(bind["att"].group, bind["att"].layer)
+            table = ctx.tables[bind["att"].group]
+            am, mx, ff = att.mixer, rec.mixer, rec.ffn
+            G = am.kv_heads
+            logits = torch.randn(rows, 16, device="cuda")
+            dn = model.blocks[3].ffn if len(model.blocks) > 3 else None
+            if name == "murutar":
+                ms = timed(lambda: rec.norm1.forward(xr, ctx))
+                kernel(f"layer norm ({label})", name, ms, gbytes=rows * d * 6 / 1e9, like="layer norm")
+                gate = torch.randn(rows, d, device="cuda")
+                follow = rec.norm2.as_following()
+                ms = timed(lambda: ops.stream_update(xr, y, rec.gate1.scale, gate=gate, **follow))
+                kernel(f"gated update + next layer norm ({label})", name, ms, gbytes=rows * d * 18 / 1e9, like="layer norm + residual + next layer norm")
+                side = rec.side
+                ms = timed(lambda: ops.stream_update(xr, y, side.norm, eps=side.eps, **follow))
+                kernel(f"rms norm + residual + next layer norm ({label})", name, ms, gbytes=rows * d * 14 / 1e9,
+                       like="layer norm + residual + next layer norm")
+                copy = h if side.reads_copy(rows) else None
+                ms = timed(lambda: side.forward(xr, copy, ctx))
+                kernel(f"token side input: gate product, table rows, projection ({label})", name, ms, gbytes=rows * d * 6 / 1e9)
+                split = mx.stack.starts[1]
+                if label == "prefill":
+                    ms = timed(lambda: ops.linear(h, mx.stack.weight[:split], None, activation="silu", out_dtype=bf))
+                    kernel(f"linear {rows}x{split}x{d} + silu (prefill)", name, ms, gflop=2.0 * rows * split * d / 1e9, like="linear + squared ReLU")
+                    qkv = torch.randn(rows, split, device="cuda").to(bf)
+                    rest = torch.randn(rows, heads * D, device="cuda")
+                    ms = timed(lambda: ops.rmsnorm_gated(ops.decay_recurrence(qkv, st, mx.powers, ctx, heads, D, D), rest, mx.norm, 1e-6, bf))
+                    kernel("lightning recurrence, 64 tokens at a time + norm and gate (prefill)", name, ms,
+                           gflop=rows * heads * (4.0 * D * D + 2 * 64 * 2 * D) / 1e9, like="mLSTM recurrence")
+                    ms = timed(lambda: ops.decay_recurrence(qkv, st, mx.powers, ctx, heads, D, D))
+                    kernel("of which the recurrence (prefill)", name, ms, gflop=rows * heads * (4.0 * D * D + 2 * 64 * 2 * D) / 1e9)
+                else:
+                    proj = torch.randn(rows, mx.stack.weight.shape[0], device="cuda")
+                    rest = proj[:, split:split + heads * D]
+                    ms = timed(lambda: ops.rmsnorm_gated(ops.decay_recurrence(proj, st, mx.powers, ctx, heads, D, D), rest, mx.norm, 1e-6, bf))
+                    kernel("lightning recurrence + norm and gate (decode)", name, ms, gbytes=batch * heads * D * D * 8 / 1e9, like="mLSTM recurrence")
+                n = am.stack.weight.shape[0]
+                ms = timed(lambda: ops.linear(h, am.stack.weight, am.stack.bias, out_dtype=f32))
+                kernel(f"linear {rows}x{n}x{d}, 32-bit out ({label})", name, ms, gflop=2.0 * rows * n * d / 1e9, like="linear, 32-bit out")
+                aproj = torch.randn(rows, n, device="cuda")
+                first = torch.randn(rows, G * D, device="cuda")
+                ms = timed(lambda: ops.rotary_prepare(aproj, kp, vp, am.rotary.freq, am.rotary.dims, ctx, table, heads, True, bf, first=first, mix=0.4))
+                kernel(f"rotation, value mix, filing ({label})", name, ms, gbytes=rows * ((heads + 2 * G) * D * 6 + G * D * 4) / 1e9,
+                       like="head norms + filing")
+                q = torch.randn(rows, heads * D, device="cuda").to(bf)
+                ms = timed(lambda: ops.grouped_attention(q, kp, vp, table, ctx, heads=heads, key_heads=G, key_dim=D, scale=am.scale,
+                                                         window=am.window, sinks=am.sinks))
+                seen = sum(min(i + 1, 512) for i in range(1024)) * 2 if label == "prefill" else batch * 512
+                if label == "prefill":
+                    kernel("windowed attention with a sink (prefill)", name, ms, gflop=seen * heads * 2 * 256 / 1e9, like="differential attention")
+                else:
+                    kernel("windowed attention with a sink + merge (decode)", name, ms, gbytes=seen * G * 2 * D * 2 / 1e9, like="differential attention")
+                scored = {"groups": 4, "keep": 2, "scores": "softmax", "group_best": 1, "normalize": False}
+                ms = timed(lambda: ops.moe_route(logits, 16, 2, scored))
+                kernel(f"routing by softmax scores in groups + plan ({label})", name, ms, like="routing by scores in groups + plan")
+                route = ops.moe_route(logits, 16, 2, scored)
+                if label == "prefill":
+                    ms = timed(lambda: ops.moe_experts_tc(h, ff.in_weight, ff.down_weight, route, activation="relu2"))
+                    kernel("experts on tcgen05: plan, gather, up with squared ReLU, down (prefill)", name, ms,
+                           gflop=2.0 * 2 * rows * 2 * ff.inner * d / 1e9, like="experts on tcgen05")
+                    picked = ops.PickedRows(*(lambda p, r: (p, route, r))(*ops.moe_experts_tc(h, ff.in_weight, ff.down_weight, route, activation="relu2")))
+                    ms = timed(lambda: ops.stream_update(xr, picked, rec.gate2.scale, gate=gate, post="copy", out_dtype=bf))
+                    kernel("experts' weighted sum + gated update + copy (prefill)", name, ms, gbytes=rows * d * 22 / 1e9, like="experts' weighted sum")
+                else:
+                    ms = timed(lambda: ops.moe_gemv(h, ff.in_weight, route, glu=None, activation="relu2"))
+                    kernel("experts' up product + squared ReLU, pair by pair (decode)", name, ms, gbytes=2 * rows * ff.inner * d * 2 / 1e9,
+                           like="experts' gate | up product")
+                if dn is not None:
+                    n = dn.stack.weight.shape[0]
+                    z = torch.randn(rows, n, device="cuda")
+                    ms = timed(lambda: ops.linear(h, dn.stack.weight, dn.stack.bias, out_dtype=f32))
+                    kernel(f"linear {rows}x{n}x{d}, 32-bit out ({label})", name, ms, gflop=2.0 * rows * n * d / 1e9, like="linear, 32-bit out")
+                    ms = timed(lambda: ops.glu_limited(z, dn.inner, 7.0, 1.702, bf))
+                    kernel(f"limited gated activation ({label})", name, ms, gbytes=rows * dn.inner * 10 / 1e9, like="gated activation")
+                    ms = timed(lambda: ops.gated_act(z, dn.inner, "gelu_tanh", bf))
+                    kernel(f"gated activation ({label})", "vedadra", ms, gbytes=rows * dn.inner * 10 / 1e9)
+                lg = torch.randn(batch, vocab, device="cuda")
+                ms = timed(lambda: ops.softcap_(lg, 30.0))
+                if label == "decode":
+                    kernel("soft cap of the logits (decode)", name, ms, gbytes=batch * vocab * 8 / 1e9)
+            else:
+                ms = timed(lambda: rec.norm1.forward(xr, ctx))
+                kernel(f"layer norm ({label})", name, ms, gbytes=rows * d * 6 / 1e9)
+                ms = timed(lambda: rec.norm1b.add_normed_then(xr, y, rec.norm2))
+                kernel(f"layer norm + residual + next layer norm ({label})", name, ms, gbytes=rows * d * 14 / 1e9)
+                proj = torch.randn(rows, mx.in_weight.shape[0], device="cuda")
+                ms = timed(lambda: ops.mlstm(proj, st, mx.norm_weight, ctx, heads, D, D, mx.cap, 1e-6, bf))
+                if label == "prefill":
+                    kernel("mLSTM recurrence, 16 tokens at a time + norm and gate (prefill)", name, ms,
+                           gflop=rows * heads * (4.0 * D * D + 2 * 16 * 2 * D) / 1e9)
+                else:
+                    kernel("mLSTM recurrence + norm and gate (decode)", name, ms, gbytes=batch * heads * D * D * 8 / 1e9)
+                n = am.in_weight.shape[0]
+                ms = timed(lambda: ops.linear(h, am.in_weight, None, out_dtype=f32))
+                kernel(f"linear {rows}x{n}x{d}, 32-bit out ({label})", name, ms, gflop=2.0 * rows * n * d / 1e9)
+                aproj = torch.randn(rows, n, device="cuda")
+                ms = timed(lambda: ops.head_norm_prepare(aproj, kp, vp, am.q_norm, am.k_norm, ctx, table, heads, G, D, 2, (heads + G) * 2 * D,
+                                                         1e-6, True, bf))
+                kernel(f"head norms + filing of keys and values ({label})", name, ms, gbytes=rows * (2 * heads + 3 * G) * D * 6 / 1e9)
+                q = torch.randn(rows, 2 * heads * D, device="cuda").to(bf)
+                hgate = aproj[:, (heads + G) * 2 * D + G * D:]
+                ms = timed(lambda: ops.grouped_attention(q, kp, vp, table, ctx, heads=2 * heads, key_heads=2 * G, key_dim=D, scale=am.scale,
+                                                         maps=2, lam=am.lam, post_scale=0.4, eps=1e-6, chunk=am.chunk, gate=hgate))
+                if label == "prefill":
+                    kernel("differential attention in chunks of 512 + finish (prefill)", name, ms, gflop=4 * (512 * 513 // 2) * 2 * heads * 2 * 256 / 1e9)
+                else:
+                    kernel("differential attention in chunks of 512 + finish (decode)", name, ms,
+                           gbytes=batch * ((ctx_len % 512) + 1) * G * 3 * D * 2 / 1e9)
+                scored = {"correction": ff.correction, "groups": 4, "keep": 2, "factor": 2.5}
+                ms = timed(lambda: ops.moe_route(logits, 16, 2, scored))
+                kernel(f"routing by scores in groups + plan ({label})", name, ms)
+                route = ops.moe_route(logits, 16, 2, scored)
+                if label == "prefill":
+                    ms = timed(lambda: ops.moe_experts_tc(h, ff.in_weight, ff.down_weight, route, float("inf"), 1.0, 0.0))
+                    kernel("experts on tcgen05: plan, gather, gate | up, silu gating, down (prefill)", name, ms,
+                           gflop=2.0 * 2 * rows * 3 * width * d / 1e9)
+                    picked, where = ops.moe_experts_tc(h, ff.in_weight, ff.down_weight, route, float("inf"), 1.0, 0.0)
+                    shared = torch.randn(rows, d, device="cuda")
+                    ms = timed(lambda: ops.moe_combine(picked, route, shared, None, where))
+                    kernel("experts' weighted sum (prefill)", name, ms, gbytes=rows * d * 16 / 1e9)
+                else:
+                    ms = timed(lambda: ops.moe_gemv(h, ff.in_weight, route, glu=(float("inf"), 1.0, 0.0)))
+                    kernel("experts' gate | up product + silu gating, pair by pair (decode)", name, ms, gbytes=2 * rows * 2 * width * d * 2 / 1e9)
+                if dn is not None:
+                    ms = timed(lambda: ops.linear(h, dn.up_weight, None, activation="relu2", out_dtype=bf))
+                    kernel(f"linear {rows}x{dn.inner}x{d} + squared ReLU ({label})", name, ms, gflop=2.0 * rows * dn.inner * d / 1e9)
+            cache.rollback(res)
+            for sl in slots:
+                cache.close(sl)
+        del engine, model
+        torch.cuda.empty_cache()
+    result["kernels"] = kernels
+    result["peaks"] = {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk["source"]}
+    return result
+
+
 def reference_line(args) -> dict:
     """The reference arm: same shape, batch, prompt length and step counts, the reference's own engine."""
     sys.path.insert(0, os.path.join(ROOT, "baseline"))
@@ -1421,8 +1703,8 @@ def main() -> int:
     parser.add_argument("--impl", default="ours", choices=("ours", "reference"))
     parser.add_argument("--no-graph", action="store_true", help="run decode steps eagerly")
     parser.add_argument("--no-points", action="store_true", help="only the decode steps at --batch")
-    parser.add_argument("--widths", default="1024,2048", help="with --only rakalix, luporax, vedadra or tesozen: the model widths to measure")
-    parser.add_argument("--only", default=None, choices=("prefill", "small", "large", "products", "rakalix", "luporax", "vedadra", "tesozen"),
+    parser.add_argument("--widths", default="1024,2048", help="with --only rakalix, luporax, vedadra, tesozen or murutar: the model widths to measure")
+    parser.add_argument("--only", default=None, choices=("prefill", "small", "large", "products", "rakalix", "luporax", "vedadra", "tesozen", "murutar"),
                         help="run one workload alone and print its numbers (for profiling): the 2,048-token prefill "
                              "step, the small shape's continuous batching, the large shape's mixed steps, or the four "
                              "products of an XL layer over row counts beside the library's matmul")
@@ -1464,6 +1746,11 @@ def main() -> int:
         for width in (int(w) for w in args.widths.split(",")):
             layers = 4 if args.layers == XL["n_layer"] else args.layers
             print(json.dumps({"tesozen_beside_luporax": run_tesozen(width, layers, args.batch, args.steps, args.warmup, pk)}), flush=True)
+        return 0
+    if args.only == "murutar":
+        for width in (int(w) for w in args.widths.split(",")):
+            layers = args.layers if args.layers != XL["n_layer"] else 4
+            print(json.dumps({"murutar_beside_tesozen": run_murutar(width, layers, args.batch, args.steps, args.warmup, pk)}), flush=True)
         return 0
     if args.only == "products":
         for row in run_products():

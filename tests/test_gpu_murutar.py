@@ -558,7 +558,8 @@ def test_lightning_remembers_far_tokens():
 
 @pytest.mark.parametrize("H,D,Dv", [(2, 16, 24), (3, 64, 128), (2, 40, 33), (1, 128, 128), (2, 7, 70)])
 def test_the_two_kernels_of_the_recurrence_against_one_another(H, D, Dv):
-    """Chunks of 64 tokens on the tensor cores (blocks of 16 and of 32 value columns) and token by token: the same inputs
+    """Chunks of 64 tokens on the tensor cores (one after the other in blocks of 16 and of 32 value columns, and side by
+    side) and token by token: the same inputs
     (exact in bfloat16), 32-bit outputs and 32-bit states, over portions that leave ragged chunks."""
     from ayaka_py_b200 import ops
     from ayaka_py_b200.cache import CacheGroupSpec
@@ -575,12 +576,15 @@ def test_the_two_kernels_of_the_recurrence_against_one_another(H, D, Dv):
     S = np.zeros((H, D, Dv))
     for t in range(300):
         S = decay[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
-    for cols in (16, 32):
+    for cols, side in ((16, False), (32, False), (0, True)):
+        if side and D * Dv % 4:
+            continue
         cache, runner = context_for([CacheGroupSpec("g", StateNeed((H, D, Dv), torch.float32), 1)], "bfloat16", max_requests=2, page_size=8, pages=8)
         got, at = [], 0
         for count in (130, 2, 63, 64, 41):
             ctx, res = step_of(cache, runner, {0: count})
-            got.append(host(ops.decay_recurrence(dev(act[at:at + count], torch.bfloat16), cache.state_layer(0, 0), powers, ctx, H, D, Dv, slice_cols=cols)))
+            got.append(host(ops.decay_recurrence(dev(act[at:at + count], torch.bfloat16), cache.state_layer(0, 0), powers, ctx, H, D, Dv, slice_cols=cols,
+                                                side_by_side=side)))
             cache.commit(res)
             at += count
         assert np.abs(np.concatenate(got) - want).max() < 1e-4 * np.abs(want).max()
