@@ -22,8 +22,8 @@
 //
 // Long portions take the chunks side by side instead of one after the other, three launches: what every chunk adds
 // to the memory, sum_s lambda^(L-1-s) k_s v_s^T, in float32 scratch (decay_chunk_sum_kernel); the walk over a
-// request's chunks, which is now a sum per cell of S and leaves every chunk's S_0 in the place of what the chunk
-// added (decay_chunk_scan_kernel); and the outputs of every chunk from its S_0 (decay_chunk_out_kernel).  The
+// request's chunks, which is now a sum per cell of S and leaves every chunk's S_0, in two bfloat16 parts, in the place of
+// what the chunk added (decay_chunk_scan_kernel); and the outputs of every chunk from its S_0 (decay_chunk_out_kernel).  The
 // arithmetic is the same.
 #include <math.h>
 
@@ -542,13 +542,14 @@ decay_chunk_sum_kernel(float* __restrict__ scratch, const __nv_bfloat16* __restr
       }
 }
 
-// Per four cells of S: the walk over a request's chunks; scratch gets every chunk's S_0, the state the last S.
+// Per eight cells of S: the walk over a request's chunks.  Scratch gets every chunk's S_0 in the place of what the chunk
+// added, as two bfloat16 parts (eight roundings, then eight remainders: the 32 bytes of the eight cells); the state the last S.
 __global__ void __launch_bounds__(128)
 decay_chunk_scan_kernel(float* __restrict__ scratch, float* __restrict__ state, const float* __restrict__ powers,
                         const int* __restrict__ req_q_start, const int* __restrict__ req_slot, int H, int cells) {
   constexpr int AHEAD = 8;
   pdl_trigger();
-  const int i = (blockIdx.x * 128 + threadIdx.x) * 4, h = blockIdx.y, r = blockIdx.z;
+  const int i = (blockIdx.x * 128 + threadIdx.x) * 8, h = blockIdx.y, r = blockIdx.z;
   int chunk0 = 0;
   for (int q = 0; q < r; ++q) chunk0 += (req_q_start[q + 1] - req_q_start[q] + DECAY_CHUNK - 1) / DECAY_CHUNK;
   const int n = req_q_start[r + 1] - req_q_start[r], chunks = (n + DECAY_CHUNK - 1) / DECAY_CHUNK;
@@ -556,26 +557,38 @@ decay_chunk_scan_kernel(float* __restrict__ scratch, float* __restrict__ state, 
   const float last = powers[h * (DECAY_CHUNK + 1) + (n - (chunks - 1) * DECAY_CHUNK)];
   pdl_wait();
   if (i >= cells) return;
-  float* S = state + ((size_t)req_slot[r] * H + h) * cells + i;
-  float4 s = *reinterpret_cast<const float4*>(S);
+  float4* S = reinterpret_cast<float4*>(state + ((size_t)req_slot[r] * H + h) * cells + i);
+  float4 s0 = S[0], s1 = S[1];
   float* at = scratch + ((size_t)chunk0 * H + h) * cells + i;
   const size_t step = (size_t)H * cells;
   for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-    float4 add[AHEAD];
+    float4 add[AHEAD][2];
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u)
-      if (c0 + u < chunks) add[u] = *reinterpret_cast<const float4*>(at + u * step);
+      if (c0 + u < chunks) {
+        add[u][0] = *reinterpret_cast<const float4*>(at + u * step);
+        add[u][1] = *reinterpret_cast<const float4*>(at + u * step + 4);
+      }
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u) {
       if (c0 + u >= chunks) break;
-      *reinterpret_cast<float4*>(at + u * step) = s;
+      uint4 hi, lo;
+      split_bf16(s0.x, s0.y, hi.x, lo.x);
+      split_bf16(s0.z, s0.w, hi.y, lo.y);
+      split_bf16(s1.x, s1.y, hi.z, lo.z);
+      split_bf16(s1.z, s1.w, hi.w, lo.w);
+      *reinterpret_cast<uint4*>(at + u * step) = hi;
+      *reinterpret_cast<uint4*>(at + u * step + 4) = lo;
       const float w = c0 + u == chunks - 1 ? last : whole;
-      s.x = fmaf(w, s.x, add[u].x); s.y = fmaf(w, s.y, add[u].y);
-      s.z = fmaf(w, s.z, add[u].z); s.w = fmaf(w, s.w, add[u].w);
+      s0.x = fmaf(w, s0.x, add[u][0].x); s0.y = fmaf(w, s0.y, add[u][0].y);
+      s0.z = fmaf(w, s0.z, add[u][0].z); s0.w = fmaf(w, s0.w, add[u][0].w);
+      s1.x = fmaf(w, s1.x, add[u][1].x); s1.y = fmaf(w, s1.y, add[u][1].y);
+      s1.z = fmaf(w, s1.z, add[u][1].z); s1.w = fmaf(w, s1.w, add[u][1].w);
     }
     at += AHEAD * step;
   }
-  *reinterpret_cast<float4*>(S) = s;
+  S[0] = s0;
+  S[1] = s1;
 }
 
 __host__ __device__ inline size_t decay_out_bytes(int D, int COLS) {
@@ -611,30 +624,16 @@ decay_chunk_out_kernel(float* __restrict__ out, const float* __restrict__ scratc
   fetch_rows<THREADS>(Qs, LDK, row0 + h * D, stride, D, D16, L, vec);
   fetch_rows<THREADS>(Ks, LDK, row0 + H * D + h * D, stride, D, D16, L, vec);
   fetch_rows<THREADS>(Vs, LDV, row0 + 2 * H * D + h * DV + c0, stride, DV - c0, COLS, L, vec);
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  const float* S = scratch + ((size_t)blockIdx.z * H + h) * D * DV;
-#pragma unroll 4
-  for (int i = tid; i < D16 * (COLS / 4); i += THREADS) {
-    const int d = i / (COLS / 4), c = (i - d * (COLS / 4)) * 4;
-    float v[4] = {0.f, 0.f, 0.f, 0.f};
-    if (d < D) {
-      if (DV % 4 == 0) {
-        if (c0 + c < DV) {
-          const float4 f = *reinterpret_cast<const float4*>(S + (size_t)d * DV + c0 + c);
-          v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-        }
-      } else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (c0 + c + e < DV) v[e] = S[(size_t)d * DV + c0 + c + e];
-      }
-    }
-    uint2 hi, lo;
-    split_bf16(v[0], v[1], hi.x, lo.x);
-    split_bf16(v[2], v[3], hi.y, lo.y);
-    *reinterpret_cast<uint2*>(Sh + d * LDV + c) = hi;
-    *reinterpret_cast<uint2*>(Sl + d * LDV + c) = lo;
+  // S_0 as the scan left it: per eight cells 16 bytes of roundings and 16 of remainders
+  const float* S = scratch + ((size_t)blockIdx.z * H + h) * D * DV + c0;
+  for (int i = tid; i < D16 * NT; i += THREADS) {
+    const int d = i / NT, c = (i - d * NT) * 8;
+    const bool live = d < D && c0 + c < DV;
+    const float* src = live ? S + (size_t)d * DV + c : scratch;
+    cp_async_16(Sh + d * LDV + c, src, live);
+    cp_async_16(Sl + d * LDV + c, live ? src + 4 : src, live);
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
   const int m0 = warp * 16;
@@ -734,7 +733,7 @@ int launch_side_by_side(float* out, float* state, float* scratch, const __nv_bfl
   const int slices = (DV + NT * 8 - 1) / (NT * 8), cells = D * DV;
   ayk_launch(decay_chunk_sum_kernel<MT, NT>, dim3(slices, H, chunks), dim3(CWARPS * 32), sum_smem, stream, scratch, qkv, stride, powers,
              req_q_start, R, H, D, DV, vec);
-  ayk_launch(decay_chunk_scan_kernel, dim3((cells / 4 + 127) / 128, H, R), dim3(128), 0, stream, scratch, state, powers, req_q_start,
+  ayk_launch(decay_chunk_scan_kernel, dim3((cells / 8 + 127) / 128, H, R), dim3(128), 0, stream, scratch, state, powers, req_q_start,
              req_slot, H, cells);
   ayk_launch(decay_chunk_out_kernel<NT>, dim3(slices, H, chunks), dim3(CWARPS * 32), out_smem, stream, out, (const float*)scratch, qkv,
              stride, powers, req_q_start, R, H, D, DV, vec);
@@ -843,7 +842,7 @@ AYK_EXPORT int ayk_decay_chunk(float* out, float* state, const void* qkv, long l
 
 // Whether the form that takes a portion's chunks side by side takes these heads.
 AYK_EXPORT int ayk_decay_chunks_takes(int D, int DV) {
-  return ayk_decay_chunk_takes(D) && D * DV % 4 == 0 && decay_out_bytes(D, 64) <= 227 * 1024;
+  return ayk_decay_chunk_takes(D) && DV % 8 == 0 && decay_out_bytes(D, 64) <= 227 * 1024;
 }
 
 // The same with all chunks of the R requests side by side (three launches).  chunks: at least as many as the requests'
