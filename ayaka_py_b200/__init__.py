@@ -4,9 +4,9 @@
 __version__ = "0.1.0"
 
 from . import models, parts  # noqa: F401  (register architectures and part kinds)
-from .config import EngineConfig, GPT2Config, LuporaxConfig, MurutarConfig, RakalixConfig, TesozenConfig, VedadraConfig
+from .config import EngineConfig, GPT2Config, LuporaxConfig, MurutarConfig, RakalixConfig, TesozenConfig, TomodraConfig, VedadraConfig
 from .engine import LLM, Request, StopCriteria
 from .sampling import SamplingParams
 
 __all__ = ["LLM", "Request", "StopCriteria", "SamplingParams", "EngineConfig", "GPT2Config", "RakalixConfig", "LuporaxConfig", "VedadraConfig", "TesozenConfig",
-           "MurutarConfig", "__version__"]
+           "MurutarConfig", "TomodraConfig", "__version__"]

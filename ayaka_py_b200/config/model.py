@@ -573,3 +573,99 @@ class MurutarConfig(ModelConfig):
         return {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width,
                 "layers": [json.loads(json.dumps(layer)) for layer in self.layers], "norm": dict(self.norm),
                 "embedding": dict(self.embedding), "token_side": dict(self.token_side), "logit_softcap": self.logit_softcap}
+
+
+_TOMODRA_MIXERS = {"attention": ("heads", "kv_heads", "dim", "vdim"),
+                   "latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank")}
+
+
+@dataclass(frozen=True)
+class TomodraConfig(ModelConfig):
+    """Tomodra: ``layers`` lists the layers in order, each {"type": "attention" | "latent_attention", "mixer": its sizes
+    and constants, "mlp": {"kind": "moe", "router": {experts, top}, "expert": {ff}, "shared": {ff}} or null}.
+    ``attention``: heads, kv_heads, dim, vdim, scale, rot {dims, base[, scaling: {factor, original, fast, slow}]} and
+    mask.size (the chunk inside which keys are seen; without ``mask`` every earlier key is); ``latent_attention``: heads,
+    dim, rot_dim, vdim, kv_rank, scale, rot {dims, base}, mask.size (the window), and optionally ``kv_from``: j, the earlier
+    latent layer whose cached latent and rotated key part this one reads instead of making its own.  ``norm.eps`` and
+    ``postln_alpha`` (the factor of the stream in every sum) are the model-wide constants.  The document names the design
+    under ``architecture``.  The model has no position limit of its own."""
+
+    ARCHITECTURE: ClassVar[str] = "Tomodra"
+
+    vocab: int = 0
+    width: int = 0
+    layers: tuple = ()
+    norm: Mapping[str, Any] = dataclasses.field(default_factory=lambda: {"eps": 1e-6})
+    postln_alpha: float = 1.0
+
+    def __post_init__(self) -> None:
+        _require_int(self.vocab, "vocab")
+        _require_int(self.width, "width")
+        if not isinstance(self.layers, (list, tuple)) or not self.layers:
+            raise ConfigError("layers must be a non-empty list")
+        object.__setattr__(self, "layers", tuple(self.layers))
+        _require_number(self.norm.get("eps") if isinstance(self.norm, Mapping) else None, "norm.eps", positive=True)
+        _require_number(self.postln_alpha, "postln_alpha")
+        for i, layer in enumerate(self.layers):
+            kind = layer.get("type") if isinstance(layer, Mapping) else None
+            if kind not in _TOMODRA_MIXERS:
+                raise ConfigError(f"layers[{i}].type must be one of {sorted(_TOMODRA_MIXERS)}, got {kind!r}")
+            mixer = layer.get("mixer")
+            if not isinstance(mixer, Mapping):
+                raise ConfigError(f"layers[{i}].mixer must give the mixer's sizes")
+            for key in _TOMODRA_MIXERS[kind]:
+                _require_int(mixer.get(key), f"layers[{i}].mixer.{key}")
+            _require_number(mixer.get("scale"), f"layers[{i}].mixer.scale")
+            rot = mixer.get("rot")
+            if not isinstance(rot, Mapping):
+                raise ConfigError(f"layers[{i}].mixer.rot must give the rotation's constants")
+            dims = _require_int(rot.get("dims"), f"layers[{i}].mixer.rot.dims")
+            _require_number(rot.get("base"), f"layers[{i}].mixer.rot.base", positive=True)
+            scaling = rot.get("scaling")
+            if scaling is not None:
+                for key in ("factor", "original", "fast", "slow"):
+                    _require_number(scaling.get(key) if isinstance(scaling, Mapping) else None,
+                                    f"layers[{i}].mixer.rot.scaling.{key}", positive=True)
+            mask = mixer.get("mask")
+            if mask is not None:
+                if not isinstance(mask, Mapping):
+                    raise ConfigError(f"layers[{i}].mixer.mask must give a size")
+                _require_int(mask.get("size"), f"layers[{i}].mixer.mask.size")
+            if kind == "attention":
+                if mixer["heads"] % mixer["kv_heads"]:
+                    raise ConfigError(f"layers[{i}].mixer: {mixer['heads']} heads cannot share {mixer['kv_heads']} key/value heads")
+                if dims % 2 or dims > mixer["dim"]:
+                    raise ConfigError(f"layers[{i}].mixer.rot.dims must be even and at most dim")
+            else:
+                if dims % 2 or dims != mixer["rot_dim"]:
+                    raise ConfigError(f"layers[{i}].mixer.rot.dims must be even and equal rot_dim")
+                source = mixer.get("kv_from")
+                if source is not None:
+                    _require_int(source, f"layers[{i}].mixer.kv_from", minimum=0)
+                    theirs = self.layers[source].get("mixer") if source < i else None
+                    if theirs is None or self.layers[source]["type"] != kind or theirs.get("kv_from") is not None:
+                        raise ConfigError(f"layers[{i}].mixer.kv_from must name an earlier latent_attention layer with a latent of its own")
+                    for key in ("kv_rank", "rot_dim", "rot"):
+                        if mixer[key] != theirs[key]:
+                            raise ConfigError(f"layers[{i}].mixer.{key} differs from that of layer {source}, whose cache it reads")
+            mlp = layer.get("mlp")
+            if mlp is None:
+                continue
+            if not isinstance(mlp, Mapping) or mlp.get("kind") != "moe":
+                raise ConfigError(f"layers[{i}].mlp.kind must be 'moe' (or mlp null), got {mlp!r}")
+            router, expert, shared = mlp.get("router"), mlp.get("expert"), mlp.get("shared")
+            if not isinstance(router, Mapping) or not isinstance(expert, Mapping):
+                raise ConfigError(f"layers[{i}].mlp must give router and expert")
+            experts = _require_int(router.get("experts"), f"layers[{i}].mlp.router.experts")
+            if _require_int(router.get("top"), f"layers[{i}].mlp.router.top") > experts:
+                raise ConfigError(f"layers[{i}].mlp.router: top exceeds experts")
+            _require_int(expert.get("ff"), f"layers[{i}].mlp.expert.ff")
+            if shared is not None:
+                if not isinstance(shared, Mapping):
+                    raise ConfigError(f"layers[{i}].mlp.shared must give the shared expert's size (or be null)")
+                _require_int(shared.get("ff"), f"layers[{i}].mlp.shared.ff")
+
+    def to_dict(self) -> dict[str, Any]:
+        return {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width,
+                "layers": [json.loads(json.dumps(layer)) for layer in self.layers], "norm": dict(self.norm),
+                "postln_alpha": self.postln_alpha}

@@ -220,7 +220,7 @@ grouped_attention_kernel(GroupedArgs a) {
   const int pos0 = a.req_pos0[req] + q0;
   const int last_pos = pos0 + rows - 1;
   const int part = blockIdx.z;
-  const int base_part = a.parts_from_window ? grouped_base_part(pos0, a.window, a.part_keys) : 0;
+  const int base_part = a.parts_from_first ? grouped_base_part(pos0, a.window, a.chunk, a.part_keys) : 0;
   const int k_first = a.part_keys > 0 ? (base_part + part) * a.part_keys : 0;
   const int k_last = a.part_keys > 0 ? min(last_pos, k_first + a.part_keys - 1) : last_pos;
   if (k_first > last_pos) return;                 // the merge does not read parts beyond the context
@@ -368,7 +368,7 @@ grouped_attention_kernel(GroupedArgs a) {
 
 // ------------------------------------------------------------------ finish --
 // One block per (row, output head), one warp per map.  The parts that the row's context reaches are merged (counted
-// from key 0, or, with ``from_window`` = the window's size, from the part that holds the window's first key):
+// from key 0, or, with ``from_first``, from the part that holds the first key in the row's window or chunk):
 // the lanes take a part each for the maxima and the parts' factors exp(m_p - M), then the sums are added up
 // four parts at a time (loads that do not wait for one another); then
 //   maps == 1: out = o * sigmoid(gate) (gate null: o);
@@ -380,13 +380,13 @@ template <typename C>
 __global__ void __launch_bounds__(64)
 grouped_finish_kernel(C* __restrict__ out, const float* __restrict__ partial_o, const float* __restrict__ partial_ml,
                       const int* __restrict__ positions, int total_rows, int QH, int DV, int parts, int part_keys,
-                      int from_window, int maps, int hpg, const float* __restrict__ gate, long long gate_stride, float lambda,
+                      int from_first, int window, int chunk, int maps, int hpg, const float* __restrict__ gate, long long gate_stride, float lambda,
                       float post_scale, float eps) {
   __shared__ float other[MAX_DV];
   pdl_trigger();
   const int t = blockIdx.x, h = blockIdx.y;
   const int pos = positions[t];
-  const int base_part = from_window > 0 ? grouped_base_part(pos, from_window, part_keys) : 0;
+  const int base_part = from_first ? grouped_base_part(pos, window, chunk, part_keys) : 0;
   const int used = part_keys > 0 ? min(parts, pos / part_keys - base_part + 1) : 1;
   pdl_wait();
   const int lane = threadIdx.x & 31, m = threadIdx.x >> 5;
@@ -533,8 +533,8 @@ AYK_EXPORT void ayk_grouped_attention_tensor_cores(int on) { g_tensor_cores = on
 // q [T, QH * DK] dense, of the cache's dtype; keys [pages, page_size, KH, DK], values [pages, page_size, VH,
 // DV].  parts > 1: the context is cut into parts of part_keys keys (grid z).  With ``partial_o`` (float32
 // [parts, T, QH, DV]) and ``partial_ml`` ([parts, T, QH, 2]) the kernel leaves unnormalized sums, maxima
-// and denominators for ayk_grouped_finish; parts_from_window: part 0 of a row is the one that holds the first key of
-// its window (single rows, no kept first keys), so that the grid covers a window and not the longest context.
+// and denominators for ayk_grouped_finish; parts_from_first: part 0 of a row is the one that holds the first key of
+// its window or chunk (single rows, no kept first keys), so that the grid covers that and not the longest context.
 // sinks [QH] or null: exp(sinks[h]) more in every denominator, without a value.  Without partial buffers it writes out [T, QH * DV] itself (parts must be 1),
 // times sigmoid(gate) when ``gate`` (float32 rows of gate_stride, QH * DV used) is given.
 AYK_EXPORT int ayk_grouped_attention(void* out, float* partial_o, float* partial_ml, const void* q, const void* kcache,
@@ -542,22 +542,22 @@ AYK_EXPORT int ayk_grouped_attention(void* out, float* partial_o, float* partial
                                      const int* req_pos0, int num_req, int total_rows, int QH, int KH, int VH, int DK,
                                      int DV, int page_size, float scale, const float* slopes, const float* sinks,
                                      int window, int keep_first, int chunk, const float* gate, long long gate_stride,
-                                     int parts, int part_keys, int parts_from_window, int dtype, cudaStream_t stream) {
+                                     int parts, int part_keys, int parts_from_first, int dtype, cudaStream_t stream) {
   if (num_req == 0 || total_rows == 0) return 0;
   AYK_REQUIRE(DK >= 1 && DK <= 1024 && DV >= 1 && DV <= MAX_DV, "ayk_grouped_attention: head sizes %d / %d (keys up to 1024, values up to %d)", DK, DV, MAX_DV);
   AYK_REQUIRE(KH >= 1 && VH >= 1 && QH % KH == 0 && QH % VH == 0 && QH <= 65535,
               "ayk_grouped_attention: %d query heads cannot share %d key heads and %d value heads", QH, KH, VH);
   AYK_REQUIRE(parts >= 1 && parts <= 65535 && (parts == 1 || (partial_o && partial_ml && part_keys > 0)), "ayk_grouped_attention: bad partition");
   AYK_REQUIRE(!partial_o == !partial_ml, "ayk_grouped_attention: partial sums need both buffers");
-  AYK_REQUIRE(!parts_from_window || (parts > 1 && window > 0 && keep_first == 0 && total_rows == num_req),
-              "ayk_grouped_attention: parts are counted from a window's first key only for single rows, with a window that keeps no first keys");
+  AYK_REQUIRE(!parts_from_first || (parts > 1 && (window > 0 || chunk > 0) && keep_first == 0 && total_rows == num_req),
+              "ayk_grouped_attention: parts are counted from the first key only for single rows, with a window or chunk and no kept first keys");
   GroupedArgs a;
   a.out = out; a.partial_o = partial_o; a.partial_ml = partial_ml; a.q = q; a.kcache = kcache; a.vcache = vcache;
   a.table = table; a.table_stride = table_stride; a.req_q_start = req_q_start; a.req_pos0 = req_pos0;
   a.num_req = num_req; a.total_rows = total_rows; a.QH = QH; a.KH = KH; a.VH = VH; a.DK = DK; a.DV = DV;
   a.page_size = page_size; a.scale = scale; a.slopes = slopes; a.sinks = sinks; a.window = window; a.keep_first = keep_first; a.chunk = chunk;
   a.gate = gate; a.gate_stride = gate_stride; a.part_keys = parts > 1 ? part_keys : 0; a.parts = parts;
-  a.parts_from_window = parts_from_window;
+  a.parts_from_first = parts_from_first;
   if (dtype == AYK_DTYPE_BF16 && g_tensor_cores) {
     const int rc = ayk_grouped_attention_mma(a, stream);
     if (rc <= 0) return rc;
@@ -589,23 +589,23 @@ AYK_EXPORT int ayk_grouped_attention(void* out, float* partial_o, float* partial
 }
 
 AYK_EXPORT int ayk_grouped_finish(void* out, const float* partial_o, const float* partial_ml, const int* positions,
-                                  int total_rows, int QH, int DV, int parts, int part_keys, int from_window, int maps, int hpg,
-                                  const float* gate, long long gate_stride, float lambda, float post_scale, float eps,
+                                  int total_rows, int QH, int DV, int parts, int part_keys, int from_first, int window, int chunk,
+                                  int maps, int hpg, const float* gate, long long gate_stride, float lambda, float post_scale, float eps,
                                   int dtype, cudaStream_t stream) {
   if (total_rows == 0) return 0;
   AYK_REQUIRE(maps == 1 || maps == 2, "ayk_grouped_finish: %d maps", maps);
   AYK_REQUIRE(QH % maps == 0 && hpg >= 1 && (QH / maps) % hpg == 0 && DV <= MAX_DV, "ayk_grouped_finish: heads do not fit");
   const int pk = parts > 1 ? part_keys : 0;
-  const int fw = parts > 1 ? from_window : 0;
+  const int ff = parts > 1 ? from_first : 0;
   const int H = QH / maps;
   AYK_REQUIRE(H <= 65535, "ayk_grouped_finish: %d heads", H);
   const dim3 grid(total_rows, H), threads(32 * maps);
   if (dtype == AYK_DTYPE_F32)
     ayk_launch(grouped_finish_kernel<float>, grid, threads, 0, stream, (float*)out, partial_o, partial_ml,
-               positions, total_rows, QH, DV, parts, pk, fw, maps, hpg, gate, gate_stride, lambda, post_scale, eps);
+               positions, total_rows, QH, DV, parts, pk, ff, window, chunk, maps, hpg, gate, gate_stride, lambda, post_scale, eps);
   else if (dtype == AYK_DTYPE_BF16)
     ayk_launch(grouped_finish_kernel<__nv_bfloat16>, grid, threads, 0, stream, (__nv_bfloat16*)out,
-               partial_o, partial_ml, positions, total_rows, QH, DV, parts, pk, fw, maps, hpg, gate, gate_stride, lambda,
+               partial_o, partial_ml, positions, total_rows, QH, DV, parts, pk, ff, window, chunk, maps, hpg, gate, gate_stride, lambda,
                post_scale, eps);
   else
     return ayk_fail("ayk_grouped_finish: unknown dtype %d", dtype);

@@ -23,7 +23,7 @@ struct GroupedArgs {
   int window, keep_first;    // window <= 0: every earlier key
   int chunk;                 // > 0: only keys of the query's own run of ``chunk`` positions (runs counted from position 0)
   int parts, part_keys;      // part_keys 0: the context is not cut
-  int parts_from_window;     // the parts are counted from the one that holds the window's first key, not from key 0
+  int parts_from_first;      // the parts are counted from the one that holds the first key in the row's window or chunk, not from key 0
   float scale;
 };
 
@@ -32,9 +32,16 @@ __host__ __device__ __forceinline__ bool grouped_visible(int i, int j, int windo
   return j <= i && (window <= 0 || i - j < window || j < keep_first) && (chunk <= 0 || j >= i / chunk * chunk);
 }
 
-// The part that a row's first part (grid index 0) is, when parts are counted from its window's first key.
-__host__ __device__ __forceinline__ int grouped_base_part(int pos, int window, int part_keys) {
-  return pos >= window ? (pos - window + 1) / part_keys : 0;
+// The first key that the query at ``pos`` sees, kept first keys aside.
+__host__ __device__ __forceinline__ int grouped_first_key(int pos, int window, int chunk) {
+  const int from_window = window > 0 && pos >= window ? pos - window + 1 : 0;
+  const int from_chunk = chunk > 0 ? pos / chunk * chunk : 0;
+  return from_window > from_chunk ? from_window : from_chunk;
+}
+
+// The part that a row's first part (grid index 0) is, when parts are counted from its first visible key.
+__host__ __device__ __forceinline__ int grouped_base_part(int pos, int window, int chunk, int part_keys) {
+  return grouped_first_key(pos, window, chunk) / part_keys;
 }
 
 // Tiles of ``step`` keys from k_first on that hold a key some row of the block may see: those below
@@ -44,8 +51,7 @@ struct GroupedTiles {
   __device__ GroupedTiles(int k_first_, int k_last, int pos0, int window, int keep_first_, int step_, int chunk = 0)
       : k_first(k_first_), step(step_), keep_first(keep_first_) {
     (void)k_last;
-    int win0 = window > 0 ? max(0, pos0 - window + 1) : 0;
-    if (chunk > 0) win0 = max(win0, pos0 / chunk * chunk);
+    const int win0 = grouped_first_key(pos0, window, chunk);
     win_tile = win0 > k_first ? k_first + (win0 - k_first) / step * step : k_first;
   }
   __device__ int next(int k0) const {

@@ -73,7 +73,7 @@ grouped_attention_mma_kernel(GroupedArgs a, int page_shift, int tq, int DKP, int
   const int pos0 = a.req_pos0[req] + q0;
   const int last_pos = pos0 + tokens - 1;
   const int part = blockIdx.z;
-  const int base_part = a.parts_from_window ? grouped_base_part(pos0, a.window, a.part_keys) : 0;
+  const int base_part = a.parts_from_first ? grouped_base_part(pos0, a.window, a.chunk, a.part_keys) : 0;
   const int k_first = a.part_keys > 0 ? (base_part + part) * a.part_keys : 0;
   const int k_last = a.part_keys > 0 ? min(last_pos, k_first + a.part_keys - 1) : last_pos;
   if (k_first > last_pos) return;                   // the merge does not read parts beyond the context

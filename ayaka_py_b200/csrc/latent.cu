@@ -56,54 +56,50 @@ __global__ void rotary_kernel(T* __restrict__ x, long long x_stride, const int* 
 //   latent  = rmsnorm(down[:rank]) * w            -> latent pages (cache dtype)
 //   k_r     = turn(down[rank:])                   -> rotated-key pages
 //   q_r     = turn(q[h, dim:]) for every head     -> query[t, h, rank:]  (float32)
+// Pairs are neighbours, or with ``halves`` dimension i and i + rot_dims/2.  The row's cos and sin wait in shared memory.
 // The unrotated query parts are projected into query[t, h, :rank] by the per-head product.
 template <typename C>
 __global__ void __launch_bounds__(128)
 latent_prepare_kernel(C* __restrict__ latent_pages, C* __restrict__ rope_pages, float* __restrict__ query,
                       const float* __restrict__ proj, int proj_stride, const float* __restrict__ norm_w,
-                      const float* __restrict__ freq, float gain, int rot_dims, const int* __restrict__ row_req,
+                      const float* __restrict__ freq, float gain, int rot_dims, int halves, const int* __restrict__ row_req,
                       const int* __restrict__ positions, const int* __restrict__ table, int table_stride, int page_size,
                       int H, int dim, int rot, int rank, float eps, int writes) {
+  extern __shared__ float turn[];            // cos [rot_dims / 2], sin [rot_dims / 2]
   __shared__ float red[4];
   pdl_trigger();
   const int t = blockIdx.x;
   const int p = positions[t];
   const int page = table[(size_t)row_req[t] * table_stride + p / page_size];
+  const int half = rot_dims >> 1;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf((float)p * freq[i], &s, &c);
+    turn[i] = c * gain;
+    turn[half + i] = s * gain;
+  }
+  __syncthreads();
   pdl_wait();
   const float* row = proj + (size_t)t * proj_stride;
   const float* down = row + (size_t)H * (dim + rot);
-  const float pos = (float)p;
-  const int half = rot_dims >> 1;
   const int Dk = rank + rot;
+  // number e of a rotated part: u cos - v sin for the first of a pair (u, v), v cos + u sin for the second
+  auto turned = [&](const float* src, int e) {
+    if (e >= rot_dims) return src[e];
+    const int pair = halves ? (e < half ? e : e - half) : e >> 1;
+    const bool second = halves ? e >= half : (e & 1) != 0;
+    const int other = halves ? (second ? e - half : e + half) : e ^ 1;
+    const float s = turn[half + pair];
+    return fmaf(src[other], second ? s : -s, src[e] * turn[pair]);
+  };
   // rotated query parts
   for (int i = threadIdx.x; i < H * rot; i += blockDim.x) {
     const int h = i / rot, e = i - h * rot;
-    const float* src = row + (size_t)h * (dim + rot) + dim;
-    float val;
-    if (e < rot_dims) {
-      const int pr = e >> 1;
-      float u = src[2 * pr], v = src[2 * pr + 1];
-      turn_pair(u, v, pos * freq[pr], gain);
-      val = (e & 1) ? v : u;
-    } else {
-      val = src[e];
-    }
-    query[((size_t)t * H + h) * Dk + rank + e] = val;
+    query[((size_t)t * H + h) * Dk + rank + e] = turned(row + (size_t)h * (dim + rot) + dim, e);
   }
   if (!writes || page <= 0) return;      // a run step that reads another's cache; a padding lane
   const size_t at = (size_t)page * page_size + (p % page_size);
-  for (int e = threadIdx.x; e < rot; e += blockDim.x) {
-    float val;
-    if (e < rot_dims) {
-      const int pr = e >> 1;
-      float u = down[rank + 2 * pr], v = down[rank + 2 * pr + 1];
-      turn_pair(u, v, pos * freq[pr], gain);
-      val = (e & 1) ? v : u;
-    } else {
-      val = down[rank + e];
-    }
-    rope_pages[at * rot + e] = from_float<C>(val);
-  }
+  for (int e = threadIdx.x; e < rot; e += blockDim.x) rope_pages[at * rot + e] = from_float<C>(turned(down + rank, e));
   float s = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) s = fmaf(down[i], down[i], s);
   s = warp_sum(s);
@@ -234,7 +230,7 @@ __global__ void __launch_bounds__(AWARPS * 32)
 latent_attention_kernel(float* __restrict__ out, const float* __restrict__ query, const C* __restrict__ latent_pages,
                         const C* __restrict__ rope_pages, const int* __restrict__ table, int table_stride,
                         const int* __restrict__ req_q_start, const int* __restrict__ req_pos0, int num_req, int H, int HG,
-                        int BR, int rank, int rot, int page_size, float scale) {
+                        int BR, int rank, int rot, int page_size, float scale, int window) {
   pdl_trigger();
   pdl_wait();
   int tile = blockIdx.x, req = -1, q0 = 0, q_len = 0;
@@ -279,7 +275,8 @@ latent_attention_kernel(float* __restrict__ out, const float* __restrict__ query
   const int last_pos = pos0 + rows - 1;
   const int* my_table = table + (size_t)req * table_stride;
 
-  for (int k0 = 0; k0 <= last_pos; k0 += AKEYS) {
+  const int first_key = window > 0 ? max(0, pos0 - window + 1) : 0;      // of the block's first row
+  for (int k0 = first_key; k0 <= last_pos; k0 += AKEYS) {
     __syncthreads();
     for (int i = threadIdx.x; i < AKEYS * Dk; i += blockDim.x) {
       const int j = i / Dk, d = i - j * Dk;
@@ -316,7 +313,7 @@ latent_attention_kernel(float* __restrict__ out, const float* __restrict__ query
         s = fmaf(qv.w, kr[d + 3], s);
       }
       for (; d < Dk; ++d) s = fmaf(qr[d], kr[d], s);
-      const bool valid = page_ok && kp <= qpos;
+      const bool valid = page_ok && kp <= qpos && (window <= 0 || qpos - kp < window);
       s = valid ? s * scale : -INFINITY;
       const float m_new = fmaxf(m_run[r], warp_max(s));
       float p = 0.f, alpha = 1.f;
@@ -368,7 +365,8 @@ latent_attention_kernel(float* __restrict__ out, const float* __restrict__ query
 template <typename C, int NC>
 int launch_latent_attention(float* out, const float* query, const void* latent_pages, const void* rope_pages,
                             const int* table, int table_stride, const int* req_q_start, const int* req_pos0, int num_req,
-                            int total_rows, int H, int rank, int rot, int page_size, float scale, cudaStream_t stream) {
+                            int total_rows, int H, int rank, int rot, int page_size, float scale, int window,
+                            cudaStream_t stream) {
   const int HG = H < AQ ? H : AQ;
   const int BR = AQ / HG;
   const int Dk = rank + rot;
@@ -381,17 +379,18 @@ int launch_latent_attention(float* out, const float* query, const void* latent_p
   }
   dim3 grid(total_rows / BR + num_req, (H + HG - 1) / HG);
   ayk_launch(latent_attention_kernel<C, NC>, grid, dim3(AWARPS * 32), smem, stream, out, query, (const C*)latent_pages,
-             (const C*)rope_pages, table, table_stride, req_q_start, req_pos0, num_req, H, HG, BR, rank, rot, page_size, scale);
+             (const C*)rope_pages, table, table_stride, req_q_start, req_pos0, num_req, H, HG, BR, rank, rot, page_size, scale,
+             window);
   return ayk_check_launch("ayk_latent_attention");
 }
 
 template <typename C>
 int pick_latent_attention(float* out, const float* query, const void* latent_pages, const void* rope_pages, const int* table,
                           int table_stride, const int* req_q_start, const int* req_pos0, int num_req, int total_rows, int H,
-                          int rank, int rot, int page_size, float scale, cudaStream_t stream) {
+                          int rank, int rot, int page_size, float scale, int window, cudaStream_t stream) {
 #define AYK_LATENT(NC)                                                                                                   \
   return launch_latent_attention<C, NC>(out, query, latent_pages, rope_pages, table, table_stride, req_q_start, req_pos0, \
-                                        num_req, total_rows, H, rank, rot, page_size, scale, stream)
+                                        num_req, total_rows, H, rank, rot, page_size, scale, window, stream)
   if (rank <= 64) AYK_LATENT(2);
   if (rank <= 128) AYK_LATENT(4);
   if (rank <= 256) AYK_LATENT(8);
@@ -418,18 +417,20 @@ AYK_EXPORT int ayk_rotary(void* x, long long x_stride, const int* positions, con
 }
 
 AYK_EXPORT int ayk_latent_prepare(void* latent_pages, void* rope_pages, float* query, const float* proj, int proj_stride,
-                                  const float* norm_w, const float* freq, float gain, int rot_dims, const int* row_req,
+                                  const float* norm_w, const float* freq, float gain, int rot_dims, int halves, const int* row_req,
                                   const int* positions, const int* table, int table_stride, int page_size, int T, int H,
                                   int dim, int rot, int rank, float eps, int writes, int cache_dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   AYK_REQUIRE(rot_dims % 2 == 0 && rot_dims <= rot, "ayk_latent_prepare: %d rotated dimensions of %d", rot_dims, rot);
+  AYK_REQUIRE(rot_dims <= 8192, "ayk_latent_prepare: %d rotated dimensions", rot_dims);
+  const size_t smem = (size_t)rot_dims * sizeof(float);
   if (cache_dtype == AYK_DTYPE_F32)
-    ayk_launch(latent_prepare_kernel<float>, dim3(T), dim3(128), 0, stream, (float*)latent_pages, (float*)rope_pages, query,
-               proj, proj_stride, norm_w, freq, gain, rot_dims, row_req, positions, table, table_stride, page_size, H, dim,
+    ayk_launch(latent_prepare_kernel<float>, dim3(T), dim3(128), smem, stream, (float*)latent_pages, (float*)rope_pages, query,
+               proj, proj_stride, norm_w, freq, gain, rot_dims, halves, row_req, positions, table, table_stride, page_size, H, dim,
                rot, rank, eps, writes);
   else if (cache_dtype == AYK_DTYPE_BF16)
-    ayk_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, stream, (__nv_bfloat16*)latent_pages,
-               (__nv_bfloat16*)rope_pages, query, proj, proj_stride, norm_w, freq, gain, rot_dims, row_req, positions, table,
+    ayk_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(T), dim3(128), smem, stream, (__nv_bfloat16*)latent_pages,
+               (__nv_bfloat16*)rope_pages, query, proj, proj_stride, norm_w, freq, gain, rot_dims, halves, row_req, positions, table,
                table_stride, page_size, H, dim, rot, rank, eps, writes);
   else
     return ayk_fail("ayk_latent_prepare: unknown dtype %d", cache_dtype);
@@ -456,21 +457,21 @@ AYK_EXPORT int ayk_head_matmul(void* out, long long out_row, int out_head, const
 }
 
 // out[t, h, :rank] = softmax_j(query[t, h] . [latent_j ; rope_j] * scale) latent_j over the cached
-// positions j <= position(t) of the row's request.  query [T, H, rank + rot] and out [T, H, rank]
+// positions j <= position(t) of the row's request (window > 0: and position(t) - j < window).  query [T, H, rank + rot] and out [T, H, rank]
 // float32; pages [pages, page_size, rank] and [pages, page_size, rot] in cache_dtype.
 AYK_EXPORT int ayk_latent_attention(float* out, const float* query, const void* latent_pages, const void* rope_pages,
                                     const int* table, int table_stride, const int* req_q_start, const int* req_pos0,
-                                    int num_req, int total_rows, int H, int rank, int rot, int page_size, float scale,
+                                    int num_req, int total_rows, int H, int rank, int rot, int page_size, float scale, int window,
                                     int cache_dtype, cudaStream_t stream) {
   if (num_req == 0 || total_rows == 0) return 0;
   AYK_REQUIRE(rank >= 1 && rank <= 512, "ayk_latent_attention: latent size %d is not in [1, 512]", rank);
   AYK_REQUIRE(rot >= 0 && rank + rot <= 640, "ayk_latent_attention: key size %d exceeds 640", rank + rot);
   if (cache_dtype == AYK_DTYPE_F32)
     return pick_latent_attention<float>(out, query, latent_pages, rope_pages, table, table_stride, req_q_start, req_pos0,
-                                        num_req, total_rows, H, rank, rot, page_size, scale, stream);
+                                        num_req, total_rows, H, rank, rot, page_size, scale, window, stream);
   if (cache_dtype == AYK_DTYPE_BF16)
     return pick_latent_attention<__nv_bfloat16>(out, query, latent_pages, rope_pages, table, table_stride, req_q_start,
-                                                req_pos0, num_req, total_rows, H, rank, rot, page_size, scale, stream);
+                                                req_pos0, num_req, total_rows, H, rank, rot, page_size, scale, window, stream);
   return ayk_fail("ayk_latent_attention: unknown dtype %d", cache_dtype);
 }
 

@@ -11,7 +11,8 @@
 // A warp owns 16 pairs and RPW columns of O (accumulators in registers); when the latent is wider
 // than RPW, two warps share the pairs: each computes S for half of the tile's positions and hands it to the other.  With one row per
 // request (decoding) a block has WM = 1 and the context is cut into partitions of PART positions
-// (grid.z) whose partial results (maximum, sum, unnormalised O) a second kernel merges.
+// (grid.z) whose partial results (maximum, sum, unnormalised O) a second kernel merges.  With a window a block visits
+// the tiles from its first row's window on, and a row's partitions are counted from the one that holds its first key.
 //
 // tcgen05 is not used here: O for 128 pairs x 512 columns would fill tensor memory alone, and
 // the score tile's K extent (rank + rot up to 576) wants operands staged in more shared memory
@@ -60,7 +61,7 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
                             const __nv_bfloat16* __restrict__ latent_pages, const __nv_bfloat16* __restrict__ rope_pages,
                             const int* __restrict__ table, int table_stride, const int* __restrict__ req_q_start,
                             const int* __restrict__ req_pos0, int num_req, int H, int HG, int BR, int rank, int rot,
-                            int page_size, float scale_log2, int parts, int part_keys) {
+                            int page_size, float scale_log2, int window, int parts, int part_keys) {
   constexpr int AQ = 16 * WM;
   pdl_trigger();
   // the last tiles of a request see the most keys: they start first (blocks are handed out in order)
@@ -79,7 +80,8 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
   const int pos0 = req_pos0[req] + q0;
   const int last_pos = pos0 + rows - 1;
   const int part = blockIdx.z;
-  const int key_lo = part * part_keys;
+  const int first_key = window > 0 ? max(0, pos0 - window + 1) : 0;      // of the block's first row
+  const int key_lo = parts > 1 ? (first_key / part_keys + part) * part_keys : first_key;
   const int key_hi = parts > 1 ? min(last_pos, key_lo + part_keys - 1) : last_pos;      // inclusive
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int wm = warp % WM, cg = warp / WM;
@@ -124,12 +126,13 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
   }
 
   // this thread's two pairs: rows g and g + 8 of the warp's 16
-  int qpos[2];
+  int qpos[2], qlow[2];                      // its position and the last position that is out of its sight
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
     const int pr = wm * 16 + g + 8 * e;
     const int r = pr / HG, hh = pr - r * HG;
     qpos[e] = (r < rows && hh < heads && pr < BR * HG) ? pos0 + r : -1;
+    qlow[e] = window > 0 ? qpos[e] - window : -1;
   }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   float o[RPW / 8][4];
@@ -224,7 +227,7 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
       for (int e = 0; e < 4; ++e) {
         const int kj = j * 8 + 2 * t4 + (e & 1);
         const int which = e >> 1;
-        const bool valid = k0 + kj <= qpos[which] && cached[kj];
+        const bool valid = k0 + kj <= qpos[which] && k0 + kj > qlow[which] && cached[kj];
         s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
         m_new[which] = fmaxf(m_new[which], s[j][e]);
       }
@@ -429,7 +432,7 @@ head_matmul_mma_kernel(O* __restrict__ out, long long out_row, int out_head, con
 template <int RPW, int CG, int WM>
 int launch(float* out, float* partial, const float* query, const void* latent_pages, const void* rope_pages, const int* table,
            int table_stride, const int* req_q_start, const int* req_pos0, int num_req, int total_rows, int H, int rank, int rot,
-           int page_size, float scale, int parts, int part_keys, cudaStream_t stream) {
+           int page_size, float scale, int window, int parts, int part_keys, cudaStream_t stream) {
   constexpr int AQ = 16 * WM;
   const int HG = H < AQ ? H : AQ;
   const int BR = AQ / HG;
@@ -444,7 +447,7 @@ int launch(float* out, float* partial, const float* query, const void* latent_pa
   dim3 grid(total_rows / BR + num_req, (H + HG - 1) / HG, parts);
   ayk_launch(latent_attention_mma_kernel<RPW, CG, WM>, grid, dim3(32 * WM * CG), smem, stream, out, partial, query,
              (const __nv_bfloat16*)latent_pages, (const __nv_bfloat16*)rope_pages, table, table_stride, req_q_start, req_pos0,
-             num_req, H, HG, BR, rank, rot, page_size, scale * 1.4426950408889634f, parts, part_keys);
+             num_req, H, HG, BR, rank, rot, page_size, scale * 1.4426950408889634f, window, parts, part_keys);
   return ayk_check_launch("ayk_latent_attention_mma");
 }
 
@@ -456,11 +459,11 @@ AYK_EXPORT int ayk_latent_attention_mma_takes(int rank, int rot) {
 }
 
 // As ayk_latent_attention, bfloat16 pages.  parts > 1 (only with one row per request): the context
-// is cut into partitions of part_keys positions; partial holds T * H * parts * (rank + 2) floats.
+// (with a window: from the partition of its first key on) is cut into partitions of part_keys positions; partial holds T * H * parts * (rank + 2) floats.
 AYK_EXPORT int ayk_latent_attention_mma(float* out, float* partial, const float* query, const void* latent_pages,
                                         const void* rope_pages, const int* table, int table_stride, const int* req_q_start,
                                         const int* req_pos0, int num_req, int total_rows, int max_q_len, int H, int rank,
-                                        int rot, int page_size, float scale, int parts, int part_keys, int* launched,
+                                        int rot, int page_size, float scale, int window, int parts, int part_keys, int* launched,
                                         cudaStream_t stream) {
   if (launched) *launched = 0;
   if (num_req == 0 || total_rows == 0) return 0;
@@ -471,9 +474,9 @@ AYK_EXPORT int ayk_latent_attention_mma(float* out, float* partial, const float*
   int rc;
 #define AYK_LM(RPW, CG)                                                                                                     \
   rc = single ? launch<RPW, CG, 1>(out, partial, query, latent_pages, rope_pages, table, table_stride, req_q_start, req_pos0, \
-                                   num_req, total_rows, H, rank, rot, page_size, scale, parts, part_keys, stream)             \
+                                   num_req, total_rows, H, rank, rot, page_size, scale, window, parts, part_keys, stream)     \
               : launch<RPW, CG, 4>(out, partial, query, latent_pages, rope_pages, table, table_stride, req_q_start, req_pos0, \
-                                   num_req, total_rows, H, rank, rot, page_size, scale, parts, part_keys, stream)
+                                   num_req, total_rows, H, rank, rot, page_size, scale, window, parts, part_keys, stream)
   if (rank <= 64) { AYK_LM(64, 1); }
   else if (rank <= 128) { AYK_LM(128, 1); }
   else if (rank <= 256) { AYK_LM(256, 1); }

@@ -18,7 +18,8 @@
 // the chosen s divided by their sum, times a factor.
 //
 // The same kernel with softmax scores: s = softmax(z) over all experts; with a correction experts are ranked by
-// s + correction[e], without one by z itself (the same order, also where s underflows).  Two more things are
+// s + correction[e], without one by z itself (the same order, also where s underflows).  Sigmoid scores without a
+// correction rank by z too unless groups count by their two best.  Two more things are
 // parameters of both: a run's score may be its largest ranking score alone, and the weights may be the chosen s as they are,
 // times the factor.
 #include <math.h>
@@ -111,8 +112,10 @@ moe_route_scored_kernel(int* __restrict__ ids, float* __restrict__ weights, cons
     inv_sum = 1.0f / warp_sum(sum);
   }
   auto score = [&](int e) { return SOFTMAX ? expf(z[e] - zmax) * inv_sum : sigmoidf(z[e]); };
+  // without a correction the logits rank alike, also where scores underflow or saturate (sums of two scores need the scores)
+  const bool by_logit = !correction && (SOFTMAX || keep >= groups || group_best == 1);
   auto ranking = [&](int e) {
-    if (SOFTMAX && !correction) return z[e];
+    if (by_logit) return z[e];
     return score(e) + (correction ? correction[e] : 0.f);
   };
   unsigned allowed = 0xffffffffu;
@@ -255,16 +258,20 @@ moe_plan_padded_kernel(int* __restrict__ row_of_pair, int* __restrict__ w_rows1,
   }
 }
 
-// out[row_of_pair[p], :] = in[p / top, :], bfloat16 rows of d elements (d a multiple of 8); a warp per pair.
+// out[row_of_pair[p], :] = in[p / top, :], bfloat16 rows of d elements (d a multiple of 8); a warp per pair.  With
+// row_scale: row_scale[row_of_pair[p]] = weights[p].
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ in, long long in_stride,
-                  const int* __restrict__ row_of_pair, int P, int top, int d) {
+                  const int* __restrict__ row_of_pair, float* __restrict__ row_scale, const float* __restrict__ weights, int P,
+                  int top, int d) {
   pdl_trigger();
   pdl_wait();
   const int p = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (p >= P) return;
   const uint4* src = reinterpret_cast<const uint4*>(in + (size_t)(p / top) * in_stride);
-  uint4* dst = reinterpret_cast<uint4*>(out + (size_t)row_of_pair[p] * d);
+  const int to = row_of_pair[p];
+  uint4* dst = reinterpret_cast<uint4*>(out + (size_t)to * d);
+  if (row_scale && lane == 0) row_scale[to] = weights[p];
   for (int i = lane; i < d / 8; i += 32) dst[i] = src[i];
 }
 
@@ -272,14 +279,16 @@ moe_gather_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restri
 // out[o(s), n] = sum_k a[r(s), k] * w[expert, n, k] over the sorted rows s of a tile; w holds N_w
 // rows per expert.  GLU: w rows [0, N) are the gate, [N, 2N) the up projection, and the output is
 // the activation of the pair.  gather: r(s) = sorted[s] / top (rows of tokens), else s.  scatter:
-// o(s) = sorted[s] (the pair's own row), else s.  On the FP32 pipes with 32-bit sums.
+// o(s) = sorted[s] (the pair's own row), else s.  early: the pair's weight multiplies its products ahead of the
+// activation (null: nothing does).  On the FP32 pipes with 32-bit sums.
 constexpr int BN = 64, BK = 32;
 
 template <typename T, typename O, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(O* __restrict__ out, const T* __restrict__ a, long long a_stride, const T* __restrict__ w,
                 const int* __restrict__ sorted, const int* __restrict__ tiles, int top, int gather, int scatter, int N,
-                int N_w, int Kd, float limit, float slope, float plus, int act) {
+                int N_w, int Kd, float limit, float slope, float plus, int act, const float* __restrict__ early) {
+  __shared__ float factor[TILE_ROWS];
   __shared__ float As[BK][TILE_ROWS + 1];
   __shared__ float Bs[GLU ? 2 : 1][BK][BN + 1];
   __shared__ int a_row[TILE_ROWS], o_row[TILE_ROWS];
@@ -292,6 +301,7 @@ moe_gemm_kernel(O* __restrict__ out, const T* __restrict__ a, long long a_stride
   if (tid < TILE_ROWS) {
     const int pair = tid < rows ? sorted[s0 + tid] : -1;
     a_row[tid] = tid < rows ? (gather ? pair / top : s0 + tid) : -1;
+    factor[tid] = early && tid < rows ? early[pair] : 1.f;
     o_row[tid] = tid < rows ? (scatter ? pair : s0 + tid) : -1;
   }
   __syncthreads();
@@ -347,7 +357,8 @@ moe_gemm_kernel(O* __restrict__ out, const T* __restrict__ a, long long a_stride
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= N) continue;
-      const float v = GLU ? glu_limited(acc[0][i][j], acc[GLU ? 1 : 0][i][j], limit, slope, plus) : apply_activation(acc[0][i][j], act);
+      const float f = factor[ty * 2 + i];
+      const float v = GLU ? glu_limited(f * acc[0][i][j], f * acc[GLU ? 1 : 0][i][j], limit, slope, plus) : apply_activation(f * acc[0][i][j], act);
       out[(size_t)dst * N + n] = from_float<O>(v);
     }
   }
@@ -371,7 +382,9 @@ template <typename O, bool GLU>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long long a_stride,
                     const __nv_bfloat16* __restrict__ w, const int* __restrict__ sorted, const int* __restrict__ tiles,
-                    int top, int gather, int scatter, int N, int N_w, int Kd, float limit, float slope, float plus, int act) {
+                    int top, int gather, int scatter, int N, int N_w, int Kd, float limit, float slope, float plus, int act,
+                    const float* __restrict__ early) {
+  __shared__ float factor[TILE_ROWS];
   __shared__ __align__(16) __nv_bfloat16 As[TILE_ROWS][TLD];
   __shared__ __align__(16) __nv_bfloat16 Bs[GLU ? 2 : 1][BN][TLD];
   __shared__ int a_row[TILE_ROWS], o_row[TILE_ROWS];
@@ -384,6 +397,7 @@ moe_gemm_mma_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, lo
   if (tid < TILE_ROWS) {
     const int pair = tid < rows ? sorted[s0 + tid] : -1;
     a_row[tid] = tid < rows ? (gather ? pair / top : s0 + tid) : -1;
+    factor[tid] = early && tid < rows ? early[pair] : 1.f;
     o_row[tid] = tid < rows ? (scatter ? pair : s0 + tid) : -1;
   }
   __syncthreads();
@@ -449,6 +463,7 @@ moe_gemm_mma_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, lo
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int dst = o_row[i * 16 + gid + half * 8];
+      const float f = factor[i * 16 + gid + half * 8];
       if (dst < 0) continue;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
@@ -456,8 +471,8 @@ moe_gemm_mma_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, lo
         for (int c = 0; c < 2; ++c) {
           const int n = n0 + warp * 16 + j * 8 + tig * 2 + c;
           if (n >= N) continue;
-          const float v0 = acc[0][i][j][half * 2 + c];
-          const float v = GLU ? glu_limited(v0, acc[GLU ? 1 : 0][i][j][half * 2 + c], limit, slope, plus) : apply_activation(v0, act);
+          const float v0 = f * acc[0][i][j][half * 2 + c];
+          const float v = GLU ? glu_limited(v0, f * acc[GLU ? 1 : 0][i][j][half * 2 + c], limit, slope, plus) : apply_activation(v0, act);
           out[(size_t)dst * N + n] = from_float<O>(v);
         }
     }
@@ -487,7 +502,7 @@ template <typename O, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long long a_stride,
                 const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids, int top, int gather, int N, int N_w,
-                int Kd, float limit, float slope, float plus, int act) {
+                int Kd, float limit, float slope, float plus, int act, const float* __restrict__ early) {
   extern __shared__ __align__(16) float xs[];          // [Kd]
   pdl_trigger();
   pdl_wait();
@@ -505,6 +520,7 @@ moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long l
     *reinterpret_cast<float4*>(xs + i * 8 + 4) = hi;
   }
   __syncthreads();
+  const float factor = early ? early[pair] : 1.f;
   const __nv_bfloat16* we = w + (size_t)ids[pair] * N_w * Kd;
   const int first = blockIdx.y * GV_COLS + warp * 8;
 #pragma unroll 1
@@ -526,8 +542,8 @@ moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long l
       g0 += dot8(wa, x0, x1);
       g1 += dot8(wb, x0, x1);
     }
-    g0 = warp_sum(g0); g1 = warp_sum(g1);
-    if (GLU) { u0 = warp_sum(u0); u1 = warp_sum(u1); }
+    g0 = factor * warp_sum(g0); g1 = factor * warp_sum(g1);
+    if (GLU) { u0 = factor * warp_sum(u0); u1 = factor * warp_sum(u1); }
     if (lane == 0) {
       out[(size_t)pair * N + n0] = from_float<O>(GLU ? glu_limited(g0, u0, limit, slope, plus) : apply_activation(g0, act));
       if (two) out[(size_t)pair * N + n1] = from_float<O>(GLU ? glu_limited(g1, u1, limit, slope, plus) : apply_activation(g1, act));
@@ -536,15 +552,17 @@ moe_gemv_kernel(O* __restrict__ out, const __nv_bfloat16* __restrict__ a, long l
 }
 
 // ------------------------------------------------- activation and weighted sum --
-// out[t, c] = act(in[t, c], in[t, n + c]) for the dense (shared) expert.
+// out[t, c] = act(f in[t, c], f in[t, n + c]) for the dense (shared) expert, f = row_scale[t] (null: 1).
 template <typename I, typename O>
 __global__ void __launch_bounds__(256)
-glu_limited_kernel(O* __restrict__ out, const I* __restrict__ in, long long stride, int n, float limit, float slope, float plus) {
+glu_limited_kernel(O* __restrict__ out, const I* __restrict__ in, long long stride, int n, float limit, float slope, float plus,
+                   const float* __restrict__ row_scale) {
   pdl_trigger();
   pdl_wait();
   const I* row = in + (size_t)blockIdx.x * stride;
+  const float f = row_scale ? row_scale[blockIdx.x] : 1.f;
   for (int c = threadIdx.x; c < n; c += blockDim.x)
-    out[(size_t)blockIdx.x * n + c] = from_float<O>(glu_limited(to_float<I>(row[c]), to_float<I>(row[n + c]), limit, slope, plus));
+    out[(size_t)blockIdx.x * n + c] = from_float<O>(glu_limited(f * to_float<I>(row[c]), f * to_float<I>(row[n + c]), limit, slope, plus));
 }
 
 // The same from 32-bit or bfloat16 rows, four columns to a thread; grid (rows, column chunks).  bfloat16 results take the
@@ -561,7 +579,8 @@ __device__ __forceinline__ void load_four(const __nv_bfloat16* p, float (&v)[4])
 
 template <typename I, typename O>
 __global__ void __launch_bounds__(256)
-glu_limited_vec_kernel(O* __restrict__ out, const I* __restrict__ in, long long stride, int n, float limit, float slope, float plus) {
+glu_limited_vec_kernel(O* __restrict__ out, const I* __restrict__ in, long long stride, int n, float limit, float slope, float plus,
+                       const float* __restrict__ row_scale) {
   pdl_trigger();
   pdl_wait();
   const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
@@ -570,6 +589,11 @@ glu_limited_vec_kernel(O* __restrict__ out, const I* __restrict__ in, long long 
   float g[4], u[4];
   load_four(row + c, g);
   load_four(row + n + c, u);
+  if (row_scale) {
+    const float f = row_scale[blockIdx.x];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { g[i] *= f; u[i] *= f; }
+  }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const float a = fminf(g[i], limit), b = fminf(fmaxf(u[i], -limit), limit) + plus;
@@ -588,7 +612,7 @@ glu_limited_vec_kernel(O* __restrict__ out, const I* __restrict__ in, long long 
 }
 
 // shared[t, :] = sum_k weights[t, k] * picked[row of pair t * top + k, :] + sigmoid(mix[t]) * shared[t, :], the
-// chosen experts in the order of their choice; row_of_pair null: the pair's own number.
+// chosen experts in the order of their choice; row_of_pair null: the pair's own number; weights null: 1.
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(float* __restrict__ shared, const float* __restrict__ picked, const int* __restrict__ row_of_pair,
                    const float* __restrict__ weights, const float* __restrict__ mix, long long mix_stride, int top, int d) {
@@ -600,7 +624,7 @@ moe_combine_kernel(float* __restrict__ shared, const float* __restrict__ picked,
     float s = 0.f;
     for (int k = 0; k < top; ++k) {
       const size_t pair = (size_t)t * top + k;
-      s = fmaf(weights[pair], picked[(size_t)(row_of_pair ? row_of_pair[pair] : pair) * d + c], s);
+      s = fmaf(weights ? weights[pair] : 1.f, picked[(size_t)(row_of_pair ? row_of_pair[pair] : pair) * d + c], s);
     }
     shared[(size_t)t * d + c] = fmaf(gate, shared[(size_t)t * d + c], s);
   }
@@ -643,19 +667,19 @@ AYK_EXPORT int ayk_moe_route_scored(int* ids, float* weights, int* sorted, int* 
 }
 
 // See moe_gemm_kernel.  dtype: of a and w; out_dtype: of out (gated rows are of the operands' dtype, plain
-// products, with the activation ``act``, of that or float32).  max_tiles: the grid's first dimension.
+// products, with the activation ``act``, of that or float32).  early [pairs] or null: see moe_gemm_kernel.  max_tiles: the grid's first dimension.
 AYK_EXPORT int ayk_moe_gemm(void* out, const void* a, long long a_stride, const void* w, const int* sorted,
                             const int* tiles, int max_tiles, int top, int gather, int scatter, int N, int N_w, int Kd,
-                            int glu, float limit, float slope, float plus, int act, int dtype, int out_dtype,
+                            int glu, float limit, float slope, float plus, int act, const float* early, int dtype, int out_dtype,
                             cudaStream_t stream) {
   if (max_tiles == 0 || N == 0) return 0;
   dim3 grid(max_tiles, (N + BN - 1) / BN);
 #define AYK_MOE(T, O, G)                                                                                              \
   ayk_launch(moe_gemm_kernel<T, O, G>, grid, dim3(256), 0, stream, (O*)out, (const T*)a, a_stride, (const T*)w, sorted, \
-             tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus, act)
+             tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus, act, early)
 #define AYK_MOE_MMA(O, G)                                                                                        \
   ayk_launch(moe_gemm_mma_kernel<O, G>, grid, dim3(128), 0, stream, (O*)out, (const __nv_bfloat16*)a, a_stride, \
-             (const __nv_bfloat16*)w, sorted, tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus, act)
+             (const __nv_bfloat16*)w, sorted, tiles, top, gather, scatter, N, N_w, Kd, limit, slope, plus, act, early)
   if (dtype == AYK_DTYPE_F32) {
     AYK_REQUIRE(out_dtype == AYK_DTYPE_F32, "ayk_moe_gemm: float32 operands give float32 rows");
     if (glu) AYK_MOE(float, float, true); else AYK_MOE(float, float, false);
@@ -679,11 +703,11 @@ AYK_EXPORT int ayk_moe_gemm(void* out, const void* a, long long a_stride, const 
 }
 
 AYK_EXPORT int ayk_glu_limited(void* out, const void* in, long long stride, int T, int n, float limit, float slope, float plus,
-                               int in_dtype, int out_dtype, cudaStream_t stream) {
+                               const float* row_scale, int in_dtype, int out_dtype, cudaStream_t stream) {
   if (T == 0 || n == 0) return 0;
   if (n % 4 == 0 && stride % 4 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0 && (n + 1023) / 1024 <= 65535) {
     const dim3 grid(T, (n + 1023) / 1024);
-#define AYK_GLU(I, O) ayk_launch(glu_limited_vec_kernel<I, O>, grid, dim3(256), 0, stream, (O*)out, (const I*)in, stride, n, limit, slope, plus)
+#define AYK_GLU(I, O) ayk_launch(glu_limited_vec_kernel<I, O>, grid, dim3(256), 0, stream, (O*)out, (const I*)in, stride, n, limit, slope, plus, row_scale)
     if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_F32) AYK_GLU(float, float);
     else if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_BF16) AYK_GLU(float, __nv_bfloat16);
     else if (in_dtype == AYK_DTYPE_BF16 && out_dtype == AYK_DTYPE_BF16) AYK_GLU(__nv_bfloat16, __nv_bfloat16);
@@ -692,13 +716,13 @@ AYK_EXPORT int ayk_glu_limited(void* out, const void* in, long long stride, int 
     return ayk_check_launch("ayk_glu_limited");
   }
   if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_F32)
-    ayk_launch(glu_limited_kernel<float, float>, dim3(T), dim3(256), 0, stream, (float*)out, (const float*)in, stride, n, limit, slope, plus);
+    ayk_launch(glu_limited_kernel<float, float>, dim3(T), dim3(256), 0, stream, (float*)out, (const float*)in, stride, n, limit, slope, plus, row_scale);
   else if (in_dtype == AYK_DTYPE_F32 && out_dtype == AYK_DTYPE_BF16)
     ayk_launch(glu_limited_kernel<float, __nv_bfloat16>, dim3(T), dim3(256), 0, stream, (__nv_bfloat16*)out, (const float*)in,
-               stride, n, limit, slope, plus);
+               stride, n, limit, slope, plus, row_scale);
   else if (in_dtype == AYK_DTYPE_BF16 && out_dtype == AYK_DTYPE_BF16)
     ayk_launch(glu_limited_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(T), dim3(256), 0, stream, (__nv_bfloat16*)out,
-               (const __nv_bfloat16*)in, stride, n, limit, slope, plus);
+               (const __nv_bfloat16*)in, stride, n, limit, slope, plus, row_scale);
   else
     return ayk_fail("ayk_glu_limited: dtypes %d -> %d", in_dtype, out_dtype);
   return ayk_check_launch("ayk_glu_limited");
@@ -707,8 +731,9 @@ AYK_EXPORT int ayk_glu_limited(void* out, const void* in, long long stride, int 
 AYK_EXPORT int ayk_moe_pad_rows() { return PAD_ROWS; }
 
 // The padded plan (see moe_plan_padded_kernel) and the gathered rows: gathered [max_tiles * 128, d] bfloat16 gets
-// row p / top of ``in`` at row_of_pair[p].  Two launches.
-AYK_EXPORT int ayk_moe_plan_padded(int* row_of_pair, int* w_rows1, int* w_rows2, void* gathered, const int* ids,
+// row p / top of ``in`` at row_of_pair[p], row_scale [max_tiles * 128] (or null) weights[p].  Two launches.
+AYK_EXPORT int ayk_moe_plan_padded(int* row_of_pair, int* w_rows1, int* w_rows2, void* gathered, float* row_scale,
+                                   const float* weights, const int* ids,
                                    const void* in, long long in_stride, int T, int E, int top, int d, int n1, int n2,
                                    int max_tiles, cudaStream_t stream) {
   if (T == 0) return 0;
@@ -716,7 +741,7 @@ AYK_EXPORT int ayk_moe_plan_padded(int* row_of_pair, int* w_rows1, int* w_rows2,
   ayk_launch(moe_plan_padded_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, row_of_pair, w_rows1, w_rows2, ids,
              T * top, E, n1, n2, max_tiles);
   ayk_launch(moe_gather_kernel, dim3((T * top + 7) / 8), dim3(256), 0, stream, (__nv_bfloat16*)gathered, (const __nv_bfloat16*)in,
-             in_stride, (const int*)row_of_pair, T * top, top, d);
+             in_stride, (const int*)row_of_pair, row_scale, weights, T * top, top, d);
   return ayk_check_launch("ayk_moe_plan_padded");
 }
 
@@ -733,7 +758,8 @@ AYK_EXPORT int ayk_moe_combine(float* shared, const float* picked, const int* ro
 AYK_EXPORT int ayk_moe_gemv_takes(int Kd, long long a_stride) { return Kd % 8 == 0 && a_stride % 8 == 0 && Kd <= 12288; }
 
 AYK_EXPORT int ayk_moe_gemv(void* out, const void* a, long long a_stride, const void* w, const int* ids, int pairs, int top,
-                            int N, int N_w, int Kd, int gather, int glu, float limit, float slope, float plus, int act, int out_dtype,
+                            int N, int N_w, int Kd, int gather, int glu, float limit, float slope, float plus, int act, const float* early,
+                            int out_dtype,
                             cudaStream_t stream) {
   if (pairs == 0 || N == 0) return 0;
   AYK_REQUIRE(ayk_moe_gemv_takes(Kd, a_stride), "ayk_moe_gemv: rows of %d elements (stride %lld)", Kd, a_stride);
@@ -741,12 +767,12 @@ AYK_EXPORT int ayk_moe_gemv(void* out, const void* a, long long a_stride, const 
   const size_t smem = (size_t)Kd * sizeof(float);
   if (glu)
     ayk_launch(moe_gemv_kernel<__nv_bfloat16, true>, grid, dim3(256), smem, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)a,
-               a_stride, (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act);
+               a_stride, (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act, early);
   else if (out_dtype == AYK_DTYPE_BF16)
     ayk_launch(moe_gemv_kernel<__nv_bfloat16, false>, grid, dim3(256), smem, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)a,
-               a_stride, (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act);
+               a_stride, (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act, early);
   else
     ayk_launch(moe_gemv_kernel<float, false>, grid, dim3(256), smem, stream, (float*)out, (const __nv_bfloat16*)a, a_stride,
-               (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act);
+               (const __nv_bfloat16*)w, ids, top, gather, N, N_w, Kd, limit, slope, plus, act, early);
   return ayk_check_launch("ayk_moe_gemv");
 }

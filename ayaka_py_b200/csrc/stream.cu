@@ -4,13 +4,14 @@
 //     gate:  y * s * sigmoid(r)     a constant s per channel and a gate r per channel (columns of the product that
 //                                   read the sublayer's input)
 //     rms:   y / rms(y) * s         an RMS norm with a weight s (eps under the root)
+//   or x[t, :] = v / rms(v) * s with v = a x[t, :] + y, a constant a (the norm of the whole sum)
 //   and, from the updated row, optionally what the next sublayer reads:
 //     copy:       x in the compute dtype
 //     layer norm: (x - mean) / sqrt(mean((x - mean)^2) + eps2) * w2 (+ b2)
 //     rms norm:   x / sqrt(mean(x^2) + eps2) * w2
 //
 // y is a float32 row, or (``picked``) the weighted sum of the rows of a token's chosen experts, added up in the
-// order of their choice.  Statistics, gates and sums are 32-bit.
+// order of their choice, or both together, the row behind a gate of one number (sigmoid of ``mix``).  Statistics, gates and sums are 32-bit.
 //
 // Beside it: a table's row per token that joins the stream behind a gate made from the stream itself
 // (token_gate_kernel, token_gate_mul_kernel), and the soft cap of the logits.
@@ -20,22 +21,24 @@
 
 namespace {
 
-enum { FROM_GATE = 0, FROM_RMS = 1 };
+enum { FROM_GATE = 0, FROM_RMS = 1, FROM_SUM = 2 };
 enum { POST_NONE = 0, POST_COPY = 1, POST_LAYER = 2, POST_RMS = 3 };
 
 struct StreamArgs {
   float* x;                  // [T, d], updated in place
   void* out;                 // [T, d] of the compute dtype, or null
-  const float* y;            // [T, d], or null with picked
+  const float* y;            // [T, d]; may be null with picked
   const float* picked;       // rows of d
   const int* row_of_pair;    // null: pair p lies at row p
-  const float* pair_weight;  // [T, top]
+  const float* pair_weight;  // [T, top]; null: 1
+  const float* mix;          // y times sigmoid(mix[t * mix_stride]); null: y as it is
   const float* gate;         // rows of gate_stride
   const float* s;            // [d]
   const float* w2;           // [d]
   const float* b2;           // [d] or null
-  long long gate_stride;
+  long long gate_stride, mix_stride;
   int d, top, post;
+  float factor;              // of x in a normed sum
   float eps, eps2;
 };
 
@@ -85,6 +88,7 @@ stream_update_vec_kernel(StreamArgs a) {
   }
   pdl_wait();
   float v[NV][4], u[NV][4];
+  const float share = a.mix ? sigmoidf(a.mix[(size_t)t * a.mix_stride]) : 1.f;
 #pragma unroll
   for (int p = 0; p < NV; ++p) {
     const int c = (p * blockDim.x + threadIdx.x) * 4;
@@ -95,14 +99,18 @@ stream_update_vec_kernel(StreamArgs a) {
     if (a.picked) {
       for (int k = 0; k < a.top; ++k) {
         const size_t pair = (size_t)t * a.top + k;
-        const float w = a.pair_weight[pair];
+        const float w = a.pair_weight ? a.pair_weight[pair] : 1.f;
         float y[4];
         load4(a.picked + (size_t)(a.row_of_pair ? a.row_of_pair[pair] : pair) * d + c, y);
 #pragma unroll
         for (int i = 0; i < 4; ++i) u[p][i] = fmaf(w, y[i], u[p][i]);
       }
-    } else {
-      load4(a.y + at + c, u[p]);
+    }
+    if (a.y) {
+      float y[4];
+      load4(a.y + at + c, y);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) u[p][i] = fmaf(share, y[i], u[p][i]);
     }
     if (FROM == FROM_GATE) {
       float r[4];
@@ -122,6 +130,21 @@ stream_update_vec_kernel(StreamArgs a) {
     for (int p = 0; p < NV; ++p)
 #pragma unroll
       for (int i = 0; i < 4; ++i) v[p][i] = fmaf(u[p][i] * inv, s[p][i], v[p][i]);
+  }
+  if (FROM == FROM_SUM) {
+    float q = 0.f;
+#pragma unroll
+    for (int p = 0; p < NV; ++p)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        v[p][i] = fmaf(a.factor, v[p][i], u[p][i]);
+        q = fmaf(v[p][i], v[p][i], q);
+      }
+    const float inv = 1.0f / sqrtf(block_total(q, red[0]) / (float)d + a.eps);
+#pragma unroll
+    for (int p = 0; p < NV; ++p)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[p][i] = v[p][i] * inv * s[p][i];
   }
 #pragma unroll
   for (int p = 0; p < NV; ++p) {
@@ -170,14 +193,14 @@ stream_update_kernel(StreamArgs a) {
   const int t = blockIdx.x, d = a.d;
   const size_t at = (size_t)t * d;
   pdl_wait();
+  const float share = a.mix ? sigmoidf(a.mix[(size_t)t * a.mix_stride]) : 1.f;
   auto value = [&](int c) {
-    if (!a.picked) return a.y[at + c];
     float u = 0.f;
-    for (int k = 0; k < a.top; ++k) {
+    for (int k = 0; a.picked && k < a.top; ++k) {
       const size_t pair = (size_t)t * a.top + k;
-      u = fmaf(a.pair_weight[pair], a.picked[(size_t)(a.row_of_pair ? a.row_of_pair[pair] : pair) * d + c], u);
+      u = fmaf(a.pair_weight ? a.pair_weight[pair] : 1.f, a.picked[(size_t)(a.row_of_pair ? a.row_of_pair[pair] : pair) * d + c], u);
     }
-    return u;
+    return a.y ? fmaf(share, a.y[at + c], u) : u;
   };
   float inv = 1.f;
   if (FROM == FROM_RMS) {
@@ -185,8 +208,23 @@ stream_update_kernel(StreamArgs a) {
     for (int c = threadIdx.x; c < d; c += blockDim.x) { const float u = value(c); q = fmaf(u, u, q); }
     inv = 1.0f / sqrtf(block_total(q, red[0]) / (float)d + a.eps);
   }
+  if (FROM == FROM_SUM) {
+    float q = 0.f;
+    for (int c = threadIdx.x; c < d; c += blockDim.x) {
+      const float v = fmaf(a.factor, a.x[at + c], value(c));
+      a.x[at + c] = v;
+      q = fmaf(v, v, q);
+    }
+    inv = 1.0f / sqrtf(block_total(q, red[0]) / (float)d + a.eps);
+  }
   float sum = 0.f;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    if (FROM == FROM_SUM) {
+      const float v = a.x[at + c] * inv * a.s[c];
+      a.x[at + c] = v;
+      sum += v;
+      continue;
+    }
     const float u = value(c);
     const float v = FROM == FROM_GATE ? fmaf(u * a.s[c], sigmoidf(a.gate[(size_t)t * a.gate_stride + c]), a.x[at + c])
                                       : fmaf(u * inv, a.s[c], a.x[at + c]);
@@ -290,27 +328,29 @@ void launch_stream(const StreamArgs& a, int T, bool vec, cudaStream_t stream) {
 
 }  // namespace
 
-// See the head of the file.  from: 0 gate, 1 rms; post: 0 none, 1 copy, 2 layer norm, 3 rms norm.  Exactly one of y
-// and picked is given; picked: rows of d, top per token, pair p = t * top + k at row row_of_pair[p] (null: p) with
-// weight pair_weight[p].
+// See the head of the file.  from: 0 gate, 1 rms, 2 the norm of the sum (factor x + y); post: 0 none, 1 copy, 2 layer
+// norm, 3 rms norm.  picked: rows of d, top per token, pair p = t * top + k at row row_of_pair[p] (null: p) with weight
+// pair_weight[p] (null: 1); y, alone or beside picked, times sigmoid(mix[t * mix_stride]) (null: 1).
 AYK_EXPORT int ayk_stream_update(float* x, void* out, const float* y, const float* picked, const int* row_of_pair,
-                                 const float* pair_weight, int top, const float* gate, long long gate_stride, const float* s,
+                                 const float* pair_weight, int top, const float* mix, long long mix_stride, float factor, const float* gate, long long gate_stride, const float* s,
                                  const float* w2, const float* b2, int T, int d, int from, int post, float eps, float eps2,
                                  int out_dtype, cudaStream_t stream) {
   if (T == 0 || d == 0) return 0;
-  AYK_REQUIRE(!y != !picked && (!picked || (pair_weight && top >= 1)), "ayk_stream_update: either rows or the rows of chosen experts");
-  AYK_REQUIRE((from == FROM_GATE && gate) || from == FROM_RMS, "ayk_stream_update: unknown source %d", from);
+  AYK_REQUIRE((y || picked) && (!picked || top >= 1) && (!mix || y), "ayk_stream_update: rows, the rows of chosen experts, or both");
+  AYK_REQUIRE((from == FROM_GATE && gate) || from == FROM_RMS || from == FROM_SUM, "ayk_stream_update: unknown source %d", from);
   AYK_REQUIRE(post >= POST_NONE && post <= POST_RMS && (post == POST_NONE || out) && (post < POST_LAYER || w2),
               "ayk_stream_update: what follows (%d) needs its output and weight", post);
   AYK_REQUIRE(out_dtype == AYK_DTYPE_F32 || out_dtype == AYK_DTYPE_BF16, "ayk_stream_update: unknown dtype %d", out_dtype);
-  const StreamArgs a{x, out, y, picked, row_of_pair, pair_weight, gate, s, w2, b2, gate_stride, d, top, post, eps, eps2};
+  const StreamArgs a{x, out, y, picked, row_of_pair, pair_weight, mix, gate, s, w2, b2, gate_stride, mix_stride, d, top, post, factor, eps, eps2};
   const bool vec = d % 4 == 0 && d <= 4096 && (!gate || gate_stride % 4 == 0) &&
                    (((uintptr_t)x | (uintptr_t)out | (uintptr_t)y | (uintptr_t)picked | (uintptr_t)gate | (uintptr_t)s | (uintptr_t)w2) & 15) == 0;
   if (out_dtype == AYK_DTYPE_BF16) {
     if (from == FROM_GATE) launch_stream<__nv_bfloat16, FROM_GATE>(a, T, vec, stream);
+    else if (from == FROM_SUM) launch_stream<__nv_bfloat16, FROM_SUM>(a, T, vec, stream);
     else launch_stream<__nv_bfloat16, FROM_RMS>(a, T, vec, stream);
   } else {
     if (from == FROM_GATE) launch_stream<float, FROM_GATE>(a, T, vec, stream);
+    else if (from == FROM_SUM) launch_stream<float, FROM_SUM>(a, T, vec, stream);
     else launch_stream<float, FROM_RMS>(a, T, vec, stream);
   }
   return ayk_check_launch("ayk_stream_update");

@@ -67,24 +67,14 @@ class Model:
         self.groups: list[CacheGroupSpec] = []
         self.bindings: list[dict[str, CacheBinding]] = []
         counts: list[int] = []
+        step_needs = self._step_needs()
         for index, step in enumerate(spec.order):
-            if not 0 <= step.layer < len(self.blocks):
-                raise ValueError(f"run step {index} names layer {step.layer}, the model has {len(self.blocks)}")
-            needs = {name: part.cache_need() for name, part in self.blocks[step.layer].parts.items()}
-            needs = {name: need for name, need in needs.items() if need is not None}
             if step.cache_of is not None:
-                if not 0 <= step.cache_of < index or not self.bindings[step.cache_of]:
-                    raise ValueError(f"run step {index}: cache_of must name an earlier run step with a cache")
-                theirs = self.bindings[step.cache_of]
-                if set(theirs) != set(needs) or any(self.groups[theirs[n].group].need != needs[n] for n in needs):
-                    raise ValueError(f"run step {index} reads a cache of another geometry")
-                self.bindings.append({n: CacheBinding(b.group, b.name, b.layer, writes=False) for n, b in theirs.items()})
+                self.bindings.append({n: CacheBinding(b.group, b.name, b.layer, writes=False)
+                                      for n, b in self.bindings[step.cache_of].items()})
                 continue
             mine: dict[str, CacheBinding] = {}
-            for name, need in needs.items():
-                if not isinstance(need, (KVNeed, StateNeed)):
-                    raise TypeError(f"cache_need() of {type(self.blocks[step.layer].parts[name]).__name__} "
-                                    f"must be KVNeed, StateNeed or None")
+            for name, need in step_needs[index].items():
                 for g, group in enumerate(self.groups):
                     if group.need == need:
                         break
@@ -97,6 +87,40 @@ class Model:
             self.bindings.append(mine)
         self.groups = [CacheGroupSpec(g.name, g.need, counts[i]) for i, g in enumerate(self.groups)]
         self.loaded = False
+
+    def _step_needs(self) -> list[dict]:
+        """What each run step's caches must keep, by part name: its own needs together with those of the later run
+        steps that read its caches (which have no entry of their own that counts)."""
+        needs: list[dict] = []
+        owner: list[int] = []
+        for index, step in enumerate(self.spec.order):
+            if not 0 <= step.layer < len(self.blocks):
+                raise ValueError(f"run step {index} names layer {step.layer}, the model has {len(self.blocks)}")
+            mine = {name: part.cache_need() for name, part in self.blocks[step.layer].parts.items()}
+            mine = {name: need for name, need in mine.items() if need is not None}
+            for name, need in mine.items():
+                if not isinstance(need, (KVNeed, StateNeed)):
+                    raise TypeError(f"cache_need() of {type(self.blocks[step.layer].parts[name]).__name__} "
+                                    f"must be KVNeed, StateNeed or None")
+            needs.append(mine)
+            owner.append(index)
+            if step.cache_of is None:
+                continue
+            if not 0 <= step.cache_of < index or not needs[step.cache_of]:
+                raise ValueError(f"run step {index}: cache_of must name an earlier run step with a cache")
+            owner[index] = owner[step.cache_of]
+            kept = needs[owner[index]]
+            if set(kept) != set(mine):
+                raise ValueError(f"run step {index} reads a cache of another geometry")
+            for name, need in mine.items():
+                if isinstance(kept[name], KVNeed) and isinstance(need, KVNeed):
+                    try:
+                        kept[name] = kept[name].together(need)
+                    except ValueError as problem:
+                        raise ValueError(f"run step {index} reads a cache of another geometry: {problem}") from None
+                elif kept[name] != need:
+                    raise ValueError(f"run step {index} reads a cache of another geometry")
+        return needs
 
     # ---------------------------------------------------------------- facts --
     @property

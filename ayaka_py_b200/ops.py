@@ -450,20 +450,25 @@ def rotary(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, gain: f
 
 def latent_prepare(proj: torch.Tensor, latent_pages: torch.Tensor, rope_pages: torch.Tensor, norm_weight: torch.Tensor,
                    freq: torch.Tensor, gain: float, rot_dims: int, ctx, table: torch.Tensor, heads: int, dim: int,
-                   rot: int, rank: int, eps: float, writes: bool) -> torch.Tensor:
+                   rot: int, rank: int, eps: float, writes: bool, halves: bool = False) -> torch.Tensor:
     """From the float32 projection rows [q (heads x (dim + rot)) | down (rank + rot) | ...]: the normed
-    latent and the rotated shared key part go into their pages (unless ``writes`` is False), the
+    latent and the rotated shared key part go into their pages (unless ``writes`` is False; the rows then need no
+    down part and ``norm_weight`` may be None), the
     rotated query parts into the returned float32 query [T, heads, rank + rot] (columns rank ..);
-    its first rank columns per head are left for the per-head product."""
+    its first rank columns per head are left for the per-head product.  ``halves``: dimension i turns with
+    i + rot_dims/2, not with its neighbour."""
     lib = _ready()
-    _f32(proj, "proj"); _f32(norm_weight, "norm_weight"); _f32(freq, "freq")
+    _f32(proj, "proj"); _f32(freq, "freq")
     T = proj.shape[0]
     P = latent_pages.shape[1]
-    if proj.shape[1] < heads * (dim + rot) + rank + rot or latent_pages.dtype != rope_pages.dtype:
+    down = rank + rot if writes else 0
+    if (proj.shape[1] < heads * (dim + rot) + down or latent_pages.dtype != rope_pages.dtype
+            or (writes and _f32(norm_weight, "norm_weight").numel() != rank)):
         raise KernelError("latent_prepare: projection rows or pages do not fit")
     query = torch.empty((T, heads, rank + rot), dtype=torch.float32, device=proj.device)
     _launch(lib.ayk_latent_prepare(_ptr(latent_pages), _ptr(rope_pages), _ptr(query), _ptr(proj), ctypes.c_int(proj.stride(0)),
-                                   _ptr(norm_weight), _ptr(freq), ctypes.c_float(gain), ctypes.c_int(rot_dims),
+                                   _ptr(norm_weight if writes else None), _ptr(freq), ctypes.c_float(gain), ctypes.c_int(rot_dims),
+                                   ctypes.c_int(1 if halves else 0),
                                    _ptr(ctx.row_req), _ptr(ctx.positions), _ptr(_i32(table, "table")),
                                    ctypes.c_int(table.stride(0)), ctypes.c_int(P), ctypes.c_int(T), ctypes.c_int(heads),
                                    ctypes.c_int(dim), ctypes.c_int(rot), ctypes.c_int(rank), ctypes.c_float(eps),
@@ -503,13 +508,15 @@ def head_matmul(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch
     return out
 
 
+LATENT_WINDOW_WHOLE = 64 # a window of up to this many keys is one partition
 LATENT_PARTS = 64        # at most this many partitions of the context when every request brings one row
 
 
 def latent_attention(query: torch.Tensor, latent_pages: torch.Tensor, rope_pages: torch.Tensor, table: torch.Tensor,
-                     ctx, scale: float, tensor_cores: bool | None = None) -> torch.Tensor:
+                     ctx, scale: float, tensor_cores: bool | None = None, window: int | None = None) -> torch.Tensor:
     """Causal attention of the step's rows over cached (latent, rotated key part) pairs shared by
-    all heads: query [T, H, rank + rot] float32; returns sum_j p_j latent_j as float32 [T, H, rank].
+    all heads: query [T, H, rank + rot] float32; returns sum_j p_j latent_j as float32 [T, H, rank].  ``window``: a
+    row sees its own position and the window - 1 before it.
     bfloat16 pages whose rows are whole 16-byte pieces go through the tensor-core kernel (a decode
     step's context cut into partitions and merged); 32-bit pages and other sizes through the
     kernel on the FP32 pipes."""
@@ -527,8 +534,12 @@ def latent_attention(query: torch.Tensor, latent_pages: torch.Tensor, rope_pages
     if tensor_cores:
         parts, part_keys, partial = 1, 0, None
         if ctx.max_q_len == 1:
-            part_keys = max(32, -(-(-(-ctx.cache.max_len // LATENT_PARTS)) // 32) * 32)
-            parts = -(-ctx.cache.max_len // part_keys)
+            reach = ctx.cache.max_len if window is None else min(window, ctx.cache.max_len)
+            part_keys = max(32, -(-(-(-reach // LATENT_PARTS)) // 32) * 32)
+            parts = -(-reach // part_keys)
+            if window is not None and reach < ctx.cache.max_len:
+                # counted from the part that holds the window's first key; a short window is not cut
+                parts = -(-(reach - 1) // part_keys) + 1 if reach > LATENT_WINDOW_WHOLE else 1
             if parts > 1:
                 partial = torch.empty((T * H * parts * (rank + 2),), dtype=torch.float32, device=query.device)
         launched = ctypes.c_int(0)
@@ -536,8 +547,8 @@ def latent_attention(query: torch.Tensor, latent_pages: torch.Tensor, rope_pages
                                             _ptr(_i32(table, "table")), ctypes.c_int(table.stride(0)), _ptr(ctx.req_q_start),
                                             _ptr(ctx.req_pos0), ctypes.c_int(ctx.num_requests), ctypes.c_int(T),
                                             ctypes.c_int(ctx.max_q_len), ctypes.c_int(H), ctypes.c_int(rank), ctypes.c_int(rot),
-                                            ctypes.c_int(latent_pages.shape[1]), ctypes.c_float(scale), ctypes.c_int(parts),
-                                            ctypes.c_int(part_keys), ctypes.byref(launched), _stream())
+                                            ctypes.c_int(latent_pages.shape[1]), ctypes.c_float(scale), ctypes.c_int(window or 0),
+                                            ctypes.c_int(parts), ctypes.c_int(part_keys), ctypes.byref(launched), _stream())
         global launches
         launches += launched.value
         _check(code)
@@ -546,7 +557,7 @@ def latent_attention(query: torch.Tensor, latent_pages: torch.Tensor, rope_pages
                                      ctypes.c_int(table.stride(0)), _ptr(ctx.req_q_start), _ptr(ctx.req_pos0),
                                      ctypes.c_int(ctx.num_requests), ctypes.c_int(T), ctypes.c_int(H), ctypes.c_int(rank),
                                      ctypes.c_int(rot), ctypes.c_int(latent_pages.shape[1]), ctypes.c_float(scale),
-                                     ctypes.c_int(_tag(latent_pages.dtype)), _stream()))
+                                     ctypes.c_int(window or 0), ctypes.c_int(_tag(latent_pages.dtype)), _stream()))
     return out
 
 
@@ -834,7 +845,7 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
     sigmoid(gate).  ``maps`` == 2: the query heads are [group][map][head of the group] and the result is per
     head o1 - lam o2, divided by its root mean square (``eps`` under the root), times ``post_scale``; a
     gate then has one number per output head.  When every request brings one row the context is cut into parts that a
-    second kernel merges (with a window that keeps no first keys, the parts that a window can reach).  ``sinks``
+    second kernel merges (with a window that keeps no first keys, or a chunk, the parts that it can reach).  ``sinks``
     float32 [heads]: exp(sinks[h]) more in every denominator (a key that is always seen and has no value).
     Returns [T, heads / maps * vdim] of the pages' dtype."""
     lib = _ready()
@@ -854,14 +865,15 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
     out = torch.empty((T, out_heads * DV), dtype=q.dtype, device=q.device)
     if sinks is not None and _f32(sinks, "sinks").numel() != heads:
         raise KernelError("grouped_attention: one sink per query head")
-    span, from_window = ctx.cache.max_len, False
+    span, from_first = ctx.cache.max_len, False
     part_keys = grouped_part(span)
     parts = max(1, -(-span // part_keys)) if ctx.max_q_len == 1 else 1
-    if parts > 1 and window and not keep_first and not chunk and window < span:
-        # a row reads its window only: the parts from the one that holds the window's first key on
-        part_keys = grouped_part(window)
-        parts = -(-(window - 1) // part_keys) + 1
-        from_window = parts > 1
+    reach = min(n for n in (span, window or span, chunk or span))
+    if parts > 1 and not keep_first and reach < span:
+        # a row reads its window or chunk only: the parts from the one that holds its first key on
+        part_keys = grouped_part(reach)
+        parts = -(-(reach - 1) // part_keys) + 1
+        from_first = parts > 1
     two_steps = parts > 1 or maps > 1
     po = pml = None
     if two_steps:
@@ -875,12 +887,13 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
                                       ctypes.c_int(P), ctypes.c_float(scale), _ptr(slopes), _ptr(sinks), ctypes.c_int(window or 0),
                                       ctypes.c_int(keep_first), ctypes.c_int(chunk or 0), _ptr(None if two_steps else gate),
                                       ctypes.c_longlong(gate_stride),
-                                      ctypes.c_int(parts), ctypes.c_int(part_keys), ctypes.c_int(1 if from_window else 0),
+                                      ctypes.c_int(parts), ctypes.c_int(part_keys), ctypes.c_int(1 if from_first else 0),
                                       ctypes.c_int(_tag(q.dtype)), _stream()))
     if two_steps:
         _launch(lib.ayk_grouped_finish(_ptr(out), _ptr(po), _ptr(pml), _ptr(ctx.positions), ctypes.c_int(T), ctypes.c_int(heads),
                                        ctypes.c_int(DV), ctypes.c_int(parts), ctypes.c_int(part_keys),
-                                       ctypes.c_int(window if from_window else 0), ctypes.c_int(maps),
+                                       ctypes.c_int(1 if from_first else 0), ctypes.c_int(window or 0), ctypes.c_int(chunk or 0),
+                                       ctypes.c_int(maps),
                                        ctypes.c_int(hpg if maps > 1 else 1), _ptr(gate), ctypes.c_longlong(gate_stride),
                                        ctypes.c_float(lam), ctypes.c_float(post_scale), ctypes.c_float(eps),
                                        ctypes.c_int(_tag(q.dtype)), _stream()))
@@ -889,9 +902,12 @@ def grouped_attention(q: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
 
 def rotary_prepare(proj: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tensor, freq: torch.Tensor | None, rot_dims: int, ctx,
                    table: torch.Tensor, heads: int, writes: bool, out_dtype: torch.dtype, first: torch.Tensor | None = None,
-                   mix: float = 0.0) -> torch.Tensor:
-    """From float32 projection rows [q | k | v | ...]: the first ``rot_dims`` dimensions of every query and key head
-    rotated by the position (dimension i with i + rot_dims/2; 0: none), keys and values into their pages (unless
+                   mix: float = 0.0, gain: float = 1.0, halves: bool = True, q_norm: torch.Tensor | None = None,
+                   k_norm: torch.Tensor | None = None, eps: float = 0.0) -> torch.Tensor:
+    """From float32 projection rows [q | k | v | ...]: with ``q_norm`` and ``k_norm`` (float32 [dim], for all query and
+    all key heads) every head RMS-normed over its numbers (``eps`` under the root); the first ``rot_dims`` dimensions of
+    every query and key head rotated by the position (dimension i with i + rot_dims/2, or neighbours unless ``halves``;
+    cos and sin times ``gain``; 0: none), keys and values into their pages (unless
     ``writes`` is False), the queries returned [T, heads * dim] in ``out_dtype``.  ``first``: float32 rows as wide as a
     token's values; the values filed are (1 - mix) v + mix first."""
     lib = _ready()
@@ -905,9 +921,13 @@ def rotary_prepare(proj: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tenso
         raise KernelError("rotary_prepare: projection rows, frequencies or pages do not fit")
     if first is not None and (first.dtype != torch.float32 or first.shape != (T, v_width) or first.stride(1) != 1):
         raise KernelError("rotary_prepare: the values to mix in must be float32 rows as wide as a token's values")
+    if (q_norm is None) != (k_norm is None) or (q_norm is not None and not (_f32(q_norm, "q_norm").numel() == _f32(k_norm, "k_norm").numel() == D)):
+        raise KernelError("rotary_prepare: query and key norms come together and have a head's size")
     q = torch.empty((T, heads * D), dtype=out_dtype, device=proj.device)
     _launch(lib.ayk_rotary_prepare(_ptr(q), _ptr(kpages), _ptr(vpages), _ptr(proj), ctypes.c_longlong(proj.stride(0)),
-                                   _ptr(freq if rot_dims else None), ctypes.c_int(rot_dims), _ptr(first),
+                                   _ptr(q_norm), _ptr(k_norm), ctypes.c_float(eps),
+                                   _ptr(freq if rot_dims else None), ctypes.c_float(gain), ctypes.c_int(0 if halves else 1),
+                                   ctypes.c_int(rot_dims), _ptr(first),
                                    ctypes.c_longlong(first.stride(0) if first is not None else 0), ctypes.c_float(1.0 - mix),
                                    ctypes.c_float(mix), _ptr(ctx.row_req), _ptr(ctx.positions), _ptr(_i32(table, "table")),
                                    ctypes.c_int(table.stride(0)), ctypes.c_int(P), ctypes.c_int(T), ctypes.c_int(heads), ctypes.c_int(G),
@@ -985,10 +1005,14 @@ def rmsnorm_gated(raw: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, e
 
 class PickedRows:
     """A routed feed-forward's result before its sum: float32 rows of the (token, choice) pairs, their weights and
-    where each pair's row lies (None: in order).  ``stream_update`` adds them up on the way."""
+    where each pair's row lies (None: in order).  ``weighted`` False: the rows are added as they are.  ``shared``: float32
+    rows of an expert that runs for every token, added as well, times sigmoid(``mix``) of the row when given.
+    ``stream_update`` adds them up on the way."""
 
-    def __init__(self, rows: torch.Tensor, route: "MoeRoute", row_of_pair: torch.Tensor | None):
+    def __init__(self, rows: torch.Tensor, route: "MoeRoute", row_of_pair: torch.Tensor | None, weighted: bool = True,
+                 shared: torch.Tensor | None = None, mix: torch.Tensor | None = None):
         self.rows, self.route, self.row_of_pair = rows, route, row_of_pair
+        self.weighted, self.shared, self.mix = weighted, shared, mix
 
 
 _STREAM_POST = {"none": 0, "copy": 1, "layernorm": 2, "rmsnorm": 3}
@@ -996,31 +1020,35 @@ _STREAM_POST = {"none": 0, "copy": 1, "layernorm": 2, "rmsnorm": 3}
 
 def stream_update(x: torch.Tensor, y: "torch.Tensor | PickedRows", scale: torch.Tensor, gate: torch.Tensor | None = None,
                   eps: float = 0.0, post: str = "none", next_weight: torch.Tensor | None = None, next_bias: torch.Tensor | None = None,
-                  next_eps: float = 0.0, out_dtype: torch.dtype = torch.float32) -> torch.Tensor | None:
-    """x += y * scale * sigmoid(gate) with ``gate`` (float32 rows [T, d]), or x += rmsnorm(y) * scale without, in place on
-    the float32 residual stream.  ``post``: what the same kernel returns of the updated rows in ``out_dtype``:
+                  next_eps: float = 0.0, out_dtype: torch.dtype = torch.float32, factor: float | None = None) -> torch.Tensor | None:
+    """x += y * scale * sigmoid(gate) with ``gate`` (float32 rows [T, d]), x = rmsnorm(factor * x + y) * scale with
+    ``factor``, or x += rmsnorm(y) * scale with neither, in place on the float32 residual stream (``eps`` under the root).  ``post``: what the same kernel returns of the updated rows in ``out_dtype``:
     nothing, a copy, their layer norm or their RMS norm with ``next_weight``."""
     lib = _ready()
     _f32(x, "x"); _f32(scale, "scale")
     T, d = x.shape
-    picked = row_of_pair = weights = None
+    picked = row_of_pair = weights = mix = None
     top = 0
     if isinstance(y, PickedRows):
-        picked, row_of_pair, weights, top = _f32(y.rows, "picked"), y.row_of_pair, y.route.weights, y.route.top
+        picked, row_of_pair, weights, top, mix = _f32(y.rows, "picked"), y.row_of_pair, y.route.weights, y.route.top, y.mix
         if picked.shape[1] != d or weights.shape[0] != T or (row_of_pair is None and picked.shape[0] != T * top):
             raise KernelError("stream_update: the pairs' rows do not fit the stream")
-        y = None
-    elif _f32(y, "y").shape != x.shape:
-        raise KernelError("stream_update: y must have the stream's shape")
+        if mix is not None and (y.shared is None or mix.dtype != torch.float32 or mix.numel() != T):
+            raise KernelError("stream_update: one gate per row of the shared expert")
+        weights = weights if y.weighted else None
+        y = y.shared
+    if (y is None and picked is None) or (y is not None and _f32(y, "y").shape != x.shape) or (gate is not None and factor is not None):
+        raise KernelError("stream_update: y must have the stream's shape; a gate and a factor exclude one another")
     if scale.numel() != d or (gate is not None and (gate.dtype != torch.float32 or gate.shape != (T, d) or gate.stride(1) != 1)):
         raise KernelError("stream_update: scale or gate rows do not fit")
     if post in ("layernorm", "rmsnorm") and _f32(next_weight, "next_weight").numel() != d:
         raise KernelError("stream_update: the following norm's weight does not fit")
     out = torch.empty((T, d), dtype=out_dtype, device=x.device) if post != "none" else None
     _launch(lib.ayk_stream_update(_ptr(x), _ptr(out), _ptr(y), _ptr(picked), _ptr(row_of_pair), _ptr(weights), ctypes.c_int(top),
-                                  _ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(scale),
+                                  _ptr(mix), ctypes.c_longlong(mix.stride(0) if mix is not None else 0),
+                                  ctypes.c_float(1.0 if factor is None else factor), _ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(scale),
                                   _ptr(next_weight), _ptr(next_bias), ctypes.c_int(T), ctypes.c_int(d),
-                                  ctypes.c_int(0 if gate is not None else 1), ctypes.c_int(_STREAM_POST[post]), ctypes.c_float(eps),
+                                  ctypes.c_int(0 if gate is not None else (1 if factor is None else 2)), ctypes.c_int(_STREAM_POST[post]), ctypes.c_float(eps),
                                   ctypes.c_float(next_eps), ctypes.c_int(_tag(out_dtype)), _stream()))
     return out
 
@@ -1111,13 +1139,14 @@ def _glu(glu: tuple | None) -> tuple[float, float, float]:
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None, out_dtype: torch.dtype,
-             activation: str | None = None) -> torch.Tensor:
+             activation: str | None = None, weigh_input: bool = False) -> torch.Tensor:
     """Grouped product over the sorted pairs.  ``glu`` = (limit, slope): a holds the tokens' rows
     [T, K], w [experts, 2 N, K] gate over up, and the result is the experts' activation
     min(g, limit) sigmoid(slope g) (clamp(u) + 1) per sorted pair, [T * top, N] in ``out_dtype``.  ``activation``
     instead: a holds the tokens' rows, w [experts, N, K], the result is the activation of the product, laid out
     alike.  Neither: a holds rows per sorted pair, w [experts, N, K], and the float32 result [T * top, N] lies pair
-    by pair (token-major).  bfloat16 operands run on the tensor cores, float32 on the FP32 pipes."""
+    by pair (token-major).  ``weigh_input``: the pair's weight multiplies its row of a (in effect: the product, in
+    32-bit, ahead of the activation).  bfloat16 operands run on the tensor cores, float32 on the FP32 pipes."""
     lib = _ready()
     E, n_w, K = w.shape
     if a.dtype != w.dtype or a.shape[1] != K or a.stride(1) != 1 or not w.is_contiguous() or (glu is not None and activation is not None):
@@ -1133,7 +1162,8 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | Non
                              ctypes.c_int(route.max_tiles), ctypes.c_int(route.top), ctypes.c_int(1 if first else 0),
                              ctypes.c_int(0 if first else 1), ctypes.c_int(N), ctypes.c_int(n_w), ctypes.c_int(K),
                              ctypes.c_int(1 if glu is not None else 0), ctypes.c_float(limit), ctypes.c_float(slope),
-                             ctypes.c_float(plus), ctypes.c_int(ACTIVATIONS[activation or "none"]), ctypes.c_int(_tag(a.dtype)),
+                             ctypes.c_float(plus), ctypes.c_int(ACTIVATIONS[activation or "none"]),
+                             _ptr(route.weights if weigh_input else None), ctypes.c_int(_tag(a.dtype)),
                              ctypes.c_int(_tag(out_dtype)), _stream()))
     return out
 
@@ -1144,11 +1174,13 @@ def moe_gemv_takes(a: torch.Tensor, w: torch.Tensor) -> bool:
             and bool(_ready().ayk_moe_gemv_takes(ctypes.c_int(w.shape[2]), ctypes.c_longlong(a.stride(0)))))
 
 
-def moe_gemv(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None, activation: str | None = None) -> torch.Tensor:
+def moe_gemv(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | None, activation: str | None = None,
+             weigh_input: bool = False) -> torch.Tensor:
     """The experts' product for a handful of pairs, each pair streaming its expert's matrix on its own: no
     sorting, rows lie pair by pair (token-major).  ``glu`` = (limit, slope): a [T, K] tokens' rows, w
     [experts, 2 N, K], bfloat16 activations [T * top, N]; ``activation``: a [T, K], w [experts, N, K], bfloat16
-    activations of the product; neither: a [T * top, K], w [experts, N, K], float32 out."""
+    activations of the product; neither: a [T * top, K], w [experts, N, K], float32 out.  ``weigh_input``: as in
+    ``moe_gemm``."""
     lib = _ready()
     E, n_w, K = w.shape
     pairs = route.ids.numel()
@@ -1162,19 +1194,22 @@ def moe_gemv(a: torch.Tensor, w: torch.Tensor, route: MoeRoute, glu: tuple | Non
     _launch(lib.ayk_moe_gemv(_ptr(out), _ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), _ptr(route.ids), ctypes.c_int(pairs),
                              ctypes.c_int(route.top), ctypes.c_int(N), ctypes.c_int(n_w), ctypes.c_int(K), ctypes.c_int(1 if first else 0),
                              ctypes.c_int(1 if glu is not None else 0), ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(plus),
-                             ctypes.c_int(ACTIVATIONS[activation or "none"]), ctypes.c_int(_tag(out_dtype)), _stream()))
+                             ctypes.c_int(ACTIVATIONS[activation or "none"]), _ptr(route.weights if weigh_input else None),
+                             ctypes.c_int(_tag(out_dtype)), _stream()))
     return out
 
 
-def glu_limited(x: torch.Tensor, n: int, limit: float, slope: float, out_dtype: torch.dtype, plus: float = 1.0) -> torch.Tensor:
+def glu_limited(x: torch.Tensor, n: int, limit: float, slope: float, out_dtype: torch.dtype, plus: float = 1.0,
+                row_scale: torch.Tensor | None = None) -> torch.Tensor:
     """min(g, limit) sigmoid(slope g) (clamp(u, -limit, limit) + plus) with g = x[:, :n] and u = x[:, n:2n]
-    of float32 or bfloat16 rows; the arithmetic is 32-bit.  An infinite limit clamps nothing."""
+    of float32 or bfloat16 rows (times ``row_scale``, float32, a number per row); the arithmetic is 32-bit.  An infinite
+    limit clamps nothing."""
     lib = _ready()
-    if x.stride(1) != 1 or x.shape[1] < 2 * n:
-        raise KernelError("glu_limited: rows of at least 2 n columns")
+    if x.stride(1) != 1 or x.shape[1] < 2 * n or (row_scale is not None and _f32(row_scale, "row_scale").numel() != x.shape[0]):
+        raise KernelError("glu_limited: rows of at least 2 n columns, one scale per row")
     out = torch.empty((x.shape[0], n), dtype=out_dtype, device=x.device)
     _launch(lib.ayk_glu_limited(_ptr(out), _ptr(x), ctypes.c_longlong(x.stride(0)), ctypes.c_int(x.shape[0]), ctypes.c_int(n),
-                                ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(plus), ctypes.c_int(_tag(x.dtype)),
+                                ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(plus), _ptr(row_scale), ctypes.c_int(_tag(x.dtype)),
                                 ctypes.c_int(_tag(out_dtype)), _stream()))
     return out
 
@@ -1183,13 +1218,17 @@ MOE_TENSOR_PAIRS = 64         # (token, choice) pairs from which the experts' pr
 
 
 def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.Tensor, route: MoeRoute, limit: float = float("inf"),
-                   slope: float = 1.0, plus: float = 1.0, activation: str | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+                   slope: float = 1.0, plus: float = 1.0, activation: str | None = None,
+                   weigh_input: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
     """The experts of a step on tcgen05 (bfloat16): the pairs' rows are gathered expert by expert, every expert's
     starting at a multiple of 128 rows, and the two products run as grouped forms of the many-row kernel, each
     128-row tile against the matrix of its expert.  in_weight [experts, 2 inner, width] gate over up (or, with
     ``activation``, [experts, inner, width] and that activation in the first product's epilogue),
-    down_weight [experts, width, inner].  Returns (float32 rows [padded, width], row of every pair)."""
+    down_weight [experts, width, inner].  ``weigh_input`` (with a gate): the pair's weight multiplies both halves of the
+    first product ahead of the activation.  Returns (float32 rows [padded, width], row of every pair)."""
     lib = _ready()
+    if weigh_input and activation is not None:
+        raise KernelError("moe_experts_tc: weights in front of the activation take experts with a gate")
     E, n1, d = in_weight.shape
     inner = n1 if activation is not None else n1 // 2
     T = h.shape[0]
@@ -1200,7 +1239,9 @@ def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.
     row_of_pair = torch.empty((pairs,), dtype=torch.int32, device=dev_)
     w_rows = torch.empty((2, max_tiles), dtype=torch.int32, device=dev_)
     gathered = torch.empty((max_tiles * pad, d), dtype=torch.bfloat16, device=dev_)
-    _launch(lib.ayk_moe_plan_padded(_ptr(row_of_pair), _ptr(w_rows[0]), _ptr(w_rows[1]), _ptr(gathered), _ptr(route.ids), _ptr(h),
+    row_scale = torch.empty((max_tiles * pad,), dtype=torch.float32, device=dev_) if weigh_input else None
+    _launch(lib.ayk_moe_plan_padded(_ptr(row_of_pair), _ptr(w_rows[0]), _ptr(w_rows[1]), _ptr(gathered), _ptr(row_scale),
+                                    _ptr(route.weights if weigh_input else None), _ptr(route.ids), _ptr(h),
                                     ctypes.c_longlong(h.stride(0)), ctypes.c_int(T), ctypes.c_int(E), ctypes.c_int(route.top),
                                     ctypes.c_int(d), ctypes.c_int(n1), ctypes.c_int(d), ctypes.c_int(max_tiles), _stream()))
     global launches
@@ -1210,7 +1251,7 @@ def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.
                                             ctypes.c_int(n1), ctypes.c_int(d), ctypes.c_int(E * n1),
                                             ctypes.c_int(ACTIVATIONS[activation or "none"]), ctypes.c_int(BF16),
                                             ctypes.c_int(sm_count()), _stream()))
-    hidden = both if activation is not None else glu_limited(both, inner, limit, slope, torch.bfloat16, plus)
+    hidden = both if activation is not None else glu_limited(both, inner, limit, slope, torch.bfloat16, plus, row_scale)
     picked = torch.empty((max_tiles * pad, d), dtype=torch.float32, device=dev_)
     _launch(lib.ayk_gemm_tc_prefill_grouped(_ptr(picked), _ptr(hidden), _ptr(down_weight), _ptr(w_rows[1]), ctypes.c_int(max_tiles * pad),
                                             ctypes.c_int(d), ctypes.c_int(inner), ctypes.c_int(E * d), ctypes.c_int(ACTIVATIONS["none"]),
@@ -1219,9 +1260,9 @@ def moe_experts_tc(h: torch.Tensor, in_weight: torch.Tensor, down_weight: torch.
 
 
 def moe_combine(picked: torch.Tensor, route: MoeRoute, shared: torch.Tensor, mix: torch.Tensor | None,
-                row_of_pair: torch.Tensor | None = None) -> torch.Tensor:
-    """shared[t] = sum_k weights[t, k] picked[row of pair t * top + k] + sigmoid(mix[t]) shared[t], in place;
-    float32.  ``row_of_pair`` None: pair p lies at row p."""
+                row_of_pair: torch.Tensor | None = None, weighted: bool = True) -> torch.Tensor:
+    """shared[t] = sum_k weights[t, k] picked[row of pair t * top + k] + sigmoid(mix[t]) shared[t], in place
+    (``weighted`` False: the picked rows as they are); float32.  ``row_of_pair`` None: pair p lies at row p."""
     lib = _ready()
     _f32(picked, "picked"); _f32(shared, "shared")
     T, d = shared.shape
@@ -1229,7 +1270,7 @@ def moe_combine(picked: torch.Tensor, route: MoeRoute, shared: torch.Tensor, mix
             (mix is not None and (mix.dtype != torch.float32 or mix.numel() != T)):
         raise KernelError("moe_combine: rows do not fit")
     _launch(lib.ayk_moe_combine(_ptr(shared), _ptr(picked), _ptr(None if row_of_pair is None else _i32(row_of_pair, "row_of_pair")),
-                                _ptr(route.weights), _ptr(mix),
+                                _ptr(route.weights if weighted else None), _ptr(mix),
                                 ctypes.c_longlong(mix.stride(0) if mix is not None else 0), ctypes.c_int(T),
                                 ctypes.c_int(route.top), ctypes.c_int(d), _stream()))
     return shared

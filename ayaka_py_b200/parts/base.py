@@ -20,7 +20,7 @@ nothing else in the package changes.
 
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Callable, ClassVar
 
 import torch
@@ -97,6 +97,16 @@ class KVNeed:
     def elements_per_token(self) -> int:
         """Key and value elements that one token takes in one layer."""
         return self.kv_heads * self.head_dim + self.v_heads * self.v_dim
+
+    def together(self, other: "KVNeed") -> "KVNeed":
+        """What a cache that serves both readers must keep: pages of one geometry, the keys that either may read."""
+        mine = (self.kv_heads, self.head_dim, self.v_heads, self.v_dim)
+        theirs = (other.kv_heads, other.head_dim, other.v_heads, other.v_dim)
+        if mine != theirs:
+            raise ValueError(f"a cache of {mine} (key heads, size, value heads, size) cannot be read as {theirs}")
+        window = None if self.window is None or other.window is None else max(self.window, other.window)
+        return replace(self, window=window, keep_first=0 if window is None else max(self.keep_first, other.keep_first),
+                       chunk=self.chunk if self.chunk == other.chunk else None)
 
 
 @dataclass(frozen=True)
@@ -298,7 +308,8 @@ def pre_norm_layer(norm1: PartSpec, mixer: PartSpec, norm2: PartSpec, ffn: PartS
 class RunStep:
     """One entry of the run order.  ``layer`` indexes ``ModelSpec.layers`` (a
     layer may be named twice).  ``cache_of``: index of an earlier run step whose
-    caches this one reads instead of keeping its own.  ``add_input``: the
+    caches this one reads instead of keeping its own (pages of the same geometry; each
+    of the two may have a window or chunk of its own).  ``add_input``: the
     embedding's output (the stream as it was before the first run step) is added
     to the stream right before this run step."""
     layer: int

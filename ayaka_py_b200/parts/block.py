@@ -170,3 +170,38 @@ class GatedPreNormBlock(Block):
 
 
 register_block(GatedPreNormBlock.KIND, GatedPreNormBlock)
+
+
+class NormedSumBlock(Block):
+    """The sublayers read the stream itself (``StreamCopy``) and a norm closes every sum, the stream with a factor of its
+    own in it: x = norm1(a x + mixer(x)); x = norm2(a x + ffn(x)).  The feed-forward (with its norm) may be absent.
+    Every sum, its norm and the copy that the next sublayer reads are one kernel (``RMSNorm.sum_normed``), which also
+    adds up a routed feed-forward's rows."""
+
+    KIND = "normed_sum"
+    PARTS = ("copy", "mixer", "norm1")
+    OPTIONAL = ("ffn", "norm2")
+
+    def __init__(self, parts):
+        super().__init__(parts)
+        if ("ffn" in parts) != ("norm2" in parts):
+            raise ValueError(f"arrangement {self.KIND!r}: ffn and norm2 come together or not at all")
+
+    def opening_norm(self):
+        return self.copy
+
+    def forward(self, x, ctx, caches):
+        h = ctx.carry.pop("opened", None)
+        if h is None:
+            h = self.copy.forward(x, ctx)
+        y, norm = self.mixer.forward(h, None, ctx, caches.get("mixer")), self.norm1
+        if "ffn" in self.parts:
+            h = norm.sum_normed(x, y, self.copy, ctx)
+            y, norm = self.ffn.forward_rows(h, ctx), self.norm2
+        opened = norm.sum_normed(x, y, ctx.following, ctx)
+        if opened is not None:
+            ctx.carry["opened"] = opened
+        return x
+
+
+register_block(NormedSumBlock.KIND, NormedSumBlock)

@@ -17,9 +17,12 @@ its own run of that many positions (runs counted from position 0 of the sequence
 output is multiplied by sigmoid(W_g h)_h, one number per head, before the output projection.  The kernel sees
 2 H query heads, 2 G key heads and G value heads.
 
-``rotary_attention``: grouped queries without norms or biases; the first ``rot.dims`` dimensions of every query and
-key head turn by the position (dimension i with i + dims/2); a window; with ``sink`` = s the softmax's denominator has
-exp(s) more (one more key, always seen, that has no value).  ``value_mix``: "first" leaves the layer's values for the
+``rotary_attention``: grouped queries without biases; the first ``rot.dims`` dimensions of every query and
+key head turn by the position (dimension i with i + dims/2, or with ``rot.layout`` "interleaved" neighbours; stretched
+frequencies with ``rot.scaling``); a window, or a chunk as above; with ``sink`` = s the softmax's denominator has
+exp(s) more (one more key, always seen, that has no value), ``sink`` "learned": a number per head, a tensor of the part.
+``qk_norm_eps``: an RMS norm per head of queries and keys, before they turn, with one weight of size ``dim`` for all
+query heads and one for all key heads.  ``value_mix``: "first" leaves the layer's values for the
 later layers of the same step, "blend" files (1 - lambda) v + lambda v_first in the place of its own values v, lambda a
 tensor of the layer (``csrc/rotary_prepare.cu``).
 
@@ -172,7 +175,8 @@ class RotaryAttention(Mixer):
     FIRST_VALUES = "first_values"            # the name in ``ctx.carry``
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rot: dict | None = None,
-                 window: int | None = None, sink: float | None = None, value_mix: str | None = None,
+                 window: int | None = None, sink: float | str | None = None, value_mix: str | None = None,
+                 chunk: int | None = None, qk_norm_eps: float | None = None,
                  dtype=torch.float32, device="cuda"):
         _check_heads(heads, kv_heads, dim, vdim)
         if dim > 1024:
@@ -182,10 +186,15 @@ class RotaryAttention(Mixer):
         if value_mix not in (None, "first", "blend"):
             raise ValueError(f"value_mix {value_mix!r}: 'first', 'blend' or None")
         self.width, self.heads, self.kv_heads, self.dim, self.vdim = width, heads, kv_heads, dim, vdim
-        self.scale, self.window, self.sink, self.value_mix, self.dtype = float(scale), window, sink, value_mix, dtype
-        self.rotary = None
+        if isinstance(sink, str) and sink != "learned":
+            raise ValueError(f"sink {sink!r}: a number, 'learned' or None")
+        self.scale, self.window, self.value_mix, self.dtype = float(scale), window, value_mix, dtype
+        self.sink, self.learned_sink = (None, True) if sink == "learned" else (sink, False)
+        self.chunk, self.qk_norm_eps = chunk, qk_norm_eps
+        self.rotary = self.q_norm = self.k_norm = None
         if rot is not None:
-            self.rotary = make_part(PartSpec("rotary", {"dims": rot["dims"], "base": rot["base"], "layout": "halves"}), dtype, device)
+            self.rotary = make_part(PartSpec("rotary", {"dims": rot["dims"], "base": rot["base"], "scaling": rot.get("scaling"),
+                                                        "layout": rot.get("layout", "halves")}), dtype, device)
         self.stack = self.sinks = self.joined = None
         self.lam = 0.0
 
@@ -196,6 +205,11 @@ class RotaryAttention(Mixer):
                "out_weight": TensorDecl((d, self.heads * self.vdim), "matrix")}
         if self.value_mix is not None:
             out["mix"] = TensorDecl((), "vector")
+        if self.qk_norm_eps is not None:
+            out["q_norm"] = TensorDecl((self.dim,), "vector")
+            out["k_norm"] = TensorDecl((self.dim,), "vector")
+        if self.learned_sink:
+            out["sink"] = TensorDecl((self.heads,), "vector")
         return out
 
     def bind(self, tensors):
@@ -205,7 +219,9 @@ class RotaryAttention(Mixer):
         self._take_views()
         if self.value_mix == "blend":
             self.lam = float(self.mix)
-        if self.sink is not None:
+        if self.learned_sink:
+            self.sinks = self.sink
+        elif self.sink is not None:
             self.sinks = torch.full((self.heads,), float(self.sink), dtype=torch.float32, device=self.stack.weight.device)
 
     def _take_views(self) -> None:
@@ -218,7 +234,8 @@ class RotaryAttention(Mixer):
         return self.stack.views[-1]
 
     def cache_need(self):
-        return KVNeed(kv_heads=self.kv_heads, head_dim=self.dim, window=self.window, value_heads=self.kv_heads, value_dim=self.vdim)
+        return KVNeed(kv_heads=self.kv_heads, head_dim=self.dim, window=self.window, value_heads=self.kv_heads, value_dim=self.vdim,
+                      chunk=self.chunk)
 
     def forward(self, h, residual, ctx, cache):
         """residual + mix(h); with ``residual`` None the mixer's output alone, float32 [T, width]."""
@@ -235,9 +252,10 @@ class RotaryAttention(Mixer):
             ctx.carry[self] = proj[:, self.joined[0]:self.joined[1]]
         rot = self.rotary
         q = ops.rotary_prepare(proj, kpages, vpages, rot.freq if rot else None, rot.dims if rot else 0, ctx, table, H, cache.writes,
-                               self.dtype, first=first, mix=self.lam)
+                               self.dtype, first=first, mix=self.lam, gain=rot.gain if rot else 1.0, halves=rot is None or rot.halves,
+                               q_norm=self.q_norm, k_norm=self.k_norm, eps=self.qk_norm_eps or 0.0)
         o = ops.grouped_attention(q, kpages, vpages, table, ctx, heads=H, key_heads=G, key_dim=D, scale=self.scale,
-                                  window=self.window, sinks=self.sinks)
+                                  window=self.window, sinks=self.sinks, chunk=self.chunk)
         return ops.linear(o, self.out_weight, None, residual=residual, out_dtype=torch.float32, out=residual)
 
 

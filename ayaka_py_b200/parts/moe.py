@@ -15,7 +15,10 @@ chosen at all), and weights the chosen experts by s over their sum, times ``rout
 no limit: silu(gate) * up).  ``shared_gated`` False: the shared expert is added as it is;
 ``shared_inner`` 0: there is none.  ``router="softmax_groups"``: s = softmax(z) over all experts, experts ranked by s,
 a run's score its largest s, the weights the chosen s as they are, times ``route_scale``.  ``activation``: experts
-without a gate, y = W_down act(W_up h) (no shared expert then).
+without a gate, y = W_down act(W_up h) (no shared expert then).  ``router="sigmoid"``: s = sigmoid(z), the ``top``
+largest, the weights the chosen s as they are, times ``route_scale``.  ``weigh`` "input": the weight multiplies the
+expert's input instead of its output, y = expert(w h); W_gate and W_up are linear, so it is applied to their 32-bit
+products, ahead of the activation.
 
 The experts' matrices are kept stacked ([experts, 2 inner, width] with gate over up, and
 [experts, width, inner]); a step sorts its (token, choice) pairs by expert on the device and runs
@@ -44,11 +47,13 @@ class MoE(FeedForward):
     def __init__(self, width: int, experts: int, top: int, inner: int, limit: float | None, shared_inner: int,
                  shared_limit: float | None, router: str = "softmax", groups: int = 1, keep: int = 1,
                  route_scale: float = 1.0, slope: float = GATE_SLOPE, plus: float = 1.0, shared_gated: bool = True,
-                 activation: str | None = None, dtype=torch.float32, device="cuda"):
+                 activation: str | None = None, weigh: str = "output", dtype=torch.float32, device="cuda"):
         if not 1 <= top <= min(experts, 16):
             raise ValueError(f"top {top} of {experts} experts: the routing kernel picks 1 to 16")
-        if router not in ("softmax", "sigmoid_groups", "softmax_groups"):
-            raise ValueError(f"unknown router {router!r}; known: softmax, sigmoid_groups, softmax_groups")
+        if router not in ("softmax", "sigmoid", "sigmoid_groups", "softmax_groups"):
+            raise ValueError(f"unknown router {router!r}; known: softmax, sigmoid, sigmoid_groups, softmax_groups")
+        if weigh not in ("output", "input") or (weigh == "input" and activation is not None):
+            raise ValueError(f"weigh {weigh!r}: 'output', or 'input' for experts with a gate")
         if activation is not None and (activation not in ops.ACTIVATIONS or shared_inner):
             raise ValueError(f"experts without a gate take one of {sorted(ops.ACTIVATIONS)} and no shared expert, got {activation!r}")
         if router != "softmax" and not (1 <= keep <= groups <= 32 and experts % groups == 0 and keep * (experts // groups) >= top):
@@ -59,7 +64,7 @@ class MoE(FeedForward):
         self.shared_limit = float("inf") if shared_limit is None else float(shared_limit)
         self.router, self.groups, self.keep, self.route_scale = router, int(groups), int(keep), float(route_scale)
         self.slope, self.plus, self.shared_gated = float(slope), float(plus), bool(shared_gated) and shared_inner > 0
-        self.activation = activation
+        self.activation, self.weigh = activation, weigh
         self.correction = self.stack = self.joined = None
         # many pairs in bfloat16, rows in whole 16-byte pieces: the experts' products run on tcgen05
         self.tensor_cores = dtype == torch.bfloat16 and width % 8 == 0 and inner % 8 == 0
@@ -129,44 +134,50 @@ class MoE(FeedForward):
             scored = {"correction": self.correction, "groups": self.groups, "keep": self.keep, "factor": self.route_scale}
         if self.router == "softmax_groups":
             scored.update(scores="softmax", group_best=1, normalize=False)
+        elif self.router == "sigmoid":
+            scored.update(normalize=False)
         many = self.tensor_cores and pairs >= ops.MOE_TENSOR_PAIRS
         few = not many and self.tensor_cores and ops.moe_gemv_takes(h, self.in_weight)
         route = ops.moe_route(logits, self.experts, self.top, scored, plan=not many and not few)
         act = self.activation
         glu = (self.limit, self.slope, self.plus)
+        early = self.weigh == "input"
         if many:
-            picked, rows = ops.moe_experts_tc(h, self.in_weight, self.down_weight, route, *glu, activation=act)
+            picked, rows = ops.moe_experts_tc(h, self.in_weight, self.down_weight, route, *glu, activation=act, weigh_input=early)
             return picked, rows, route
         glu = glu if act is None else None
         if few:
             # a handful of pairs (a step of single tokens): every pair streams its expert's matrices on its own
-            hidden = ops.moe_gemv(h, self.in_weight, route, glu=glu, activation=act)
+            hidden = ops.moe_gemv(h, self.in_weight, route, glu=glu, activation=act, weigh_input=early)
             return ops.moe_gemv(hidden, self.down_weight, route, glu=None), None, route                    # [T * K, d]
-        hidden = ops.moe_gemm(h, self.in_weight, route, glu=glu, out_dtype=self.dtype, activation=act)
+        hidden = ops.moe_gemm(h, self.in_weight, route, glu=glu, out_dtype=self.dtype, activation=act, weigh_input=early)
         return ops.moe_gemm(hidden, self.down_weight, route, glu=None, out_dtype=torch.float32), None, route
 
     def forward(self, h, residual, ctx):
         """ff(h) (+ residual), float32 [T, width].  h: rows in the compute dtype."""
-        T, d = h.shape[0], self.width
         picked, rows, route = self._experts(h, ctx)
-        if self.shared_inner:
-            sp = ops.linear(h, self.shared_in, None, out_dtype=torch.float32)
-            sh = ops.glu_limited(sp, self.shared_inner, self.shared_limit, self.slope, self.dtype, self.plus)
-            shared = ops.linear(sh, self.shared_down, None, out_dtype=torch.float32)
-        else:
-            shared = torch.zeros((T, d), dtype=torch.float32, device=h.device)
-        out = ops.moe_combine(picked, route, shared, sp[:, 2 * self.shared_inner] if self.shared_gated else None, rows)
+        shared, mix = self._shared(h)
+        if shared is None:
+            shared = torch.zeros((h.shape[0], self.width), dtype=torch.float32, device=h.device)
+        out = ops.moe_combine(picked, route, shared, mix, rows, weighted=self.weigh == "output")
         if residual is not None:
             residual.add_(out)
             return residual
         return out
 
+    def _shared(self, h):
+        """The shared expert's float32 rows and the column of their gates' logits; None for what there is not."""
+        if not self.shared_inner:
+            return None, None
+        sp = ops.linear(h, self.shared_in, None, out_dtype=torch.float32)
+        sh = ops.glu_limited(sp, self.shared_inner, self.shared_limit, self.slope, self.dtype, self.plus)
+        return ops.linear(sh, self.shared_down, None, out_dtype=torch.float32), sp[:, 2 * self.shared_inner] if self.shared_gated else None
+
     def forward_rows(self, h, ctx):
-        """Without a shared expert the chosen experts' rows themselves: their sum is left to the kernel that needs it."""
-        if self.shared_inner:
-            return self.forward(h, None, ctx)
+        """The chosen experts' rows (and the shared expert's) themselves: their sum is left to the kernel that needs it."""
         picked, rows, route = self._experts(h, ctx)
-        return ops.PickedRows(picked, route, rows)
+        shared, mix = self._shared(h)
+        return ops.PickedRows(picked, route, rows, weighted=self.weigh == "output", shared=shared, mix=mix)
 
 
 register_part(MoE.KIND, MoE)

@@ -54,16 +54,16 @@ class RMSNorm(Norm):
     ``offset``: the checkpoint stores weight - offset (a weight kept around zero has offset 1); the
     sum is made once, in 32-bit, when the tensor is bound.  ``groups`` > 1: the row is cut into that
     many equal consecutive runs and each is divided by its own root mean square; the weight spans
-    the whole row."""
+    the whole row.  ``stream_factor``: the factor of the stream in ``sum_normed``."""
 
     KIND = "rmsnorm"
 
-    def __init__(self, width: int, eps: float, out_scale: float = 1.0, offset: float = 0.0, groups: int = 1,
+    def __init__(self, width: int, eps: float, out_scale: float = 1.0, offset: float = 0.0, groups: int = 1, stream_factor: float = 1.0,
                  dtype=torch.float32, device="cuda"):
         if groups < 1 or width % groups:
             raise ValueError(f"a row of {width} is not {groups} equal groups")
         self.width, self.eps, self.out_scale, self.offset = width, float(eps), float(out_scale), float(offset)
-        self.groups = int(groups)
+        self.groups, self.stream_factor = int(groups), float(stream_factor)
         self.dtype = dtype
         self.weight = None
 
@@ -89,6 +89,14 @@ class RMSNorm(Norm):
         """x += out_scale * norm(y), in place; x and y float32 [T, width]."""
         return ops.rmsnorm_residual(x, y, self.weight, self.eps, self.out_scale, groups=self.groups)
 
+    def sum_normed(self, x, y, following: Norm | None, ctx):
+        """x = norm(stream_factor * x + y), in place: a norm that closes a sum (``y`` float32 rows or
+        ``ops.PickedRows``).  Returns ``following`` of the new x (None: nothing), from the same kernel where that can be."""
+        if self.groups != 1 or self.out_scale != 1.0:
+            raise ValueError("a norm over the sum with the stream spans the whole row and has no output factor")
+        post = following.as_following() if following is not None else None
+        h = ops.stream_update(x, y, self.weight, factor=self.stream_factor, eps=self.eps, **(post or {}))
+        return following.forward(x, ctx) if following is not None and post is None else h
 
     def add_normed_then(self, x, y, following: "RMSNorm"):
         """x += out_scale * norm(y) in place, and ``following``'s norm of the updated x (one kernel when both
@@ -100,5 +108,22 @@ class RMSNorm(Norm):
                                          following.dtype, groups=self.groups)
 
 
+class StreamCopy(Norm):
+    """No norm: the stream as it is, in the compute dtype (float32: the stream itself), for sublayers that read it so."""
+
+    KIND = "stream_copy"
+
+    def __init__(self, width: int, dtype=torch.float32, device="cuda"):
+        self.width, self.dtype = width, dtype
+
+    def forward(self, x, ctx, rows=None):
+        x = x if rows is None else x[rows]
+        return x if self.dtype == torch.float32 else ops.token_shift(x, None, None, None, self.dtype)
+
+    def as_following(self):
+        return {"post": "copy", "out_dtype": self.dtype}
+
+
+register_part(StreamCopy.KIND, StreamCopy)
 register_part(LayerNorm.KIND, LayerNorm)
 register_part(RMSNorm.KIND, RMSNorm)
