@@ -109,22 +109,6 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
     }
     return;
   }
-  // the pairs' queries as bfloat16 (rank and rot are multiples of 8, so a pair's row is whole float4s;
-  // the padding columns are zeros)
-  const int quads = Dp / 4;
-#pragma unroll 4
-  for (int i = threadIdx.x; i < AQ * quads; i += blockDim.x) {
-    const int pr = i / quads, d = (i - pr * quads) * 4;
-    const int r = pr / HG, hh = pr - r * HG;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < rows && hh < heads && pr < BR * HG && d < Dk)
-      v = *reinterpret_cast<const float4*>(query + ((size_t)(row0 + r) * H + h0 + hh) * Dk + d);
-    uint2 packed;
-    packed.x = pack_bf16(v.x, v.y);
-    packed.y = pack_bf16(v.z, v.w);
-    *reinterpret_cast<uint2*>(Qs + pr * ld + d) = packed;
-  }
-
   // this thread's two pairs: rows g and g + 8 of the warp's 16
   int qpos[2], qlow[2];                      // its position and the last position that is out of its sight
 #pragma unroll
@@ -145,28 +129,54 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
   // buffers: tile i + 1 is on its way while tile i is used.
   const int chunks_lat = rank / 8, chunks_rot = rot / 8, chunks = Dp / 8;
   const int nwarps = WM * CG;
-  auto fetch = [&](int k0, __nv_bfloat16* dst, int* flags) {
+  // Lane j looks up position j of a tile (its cell in the pages, or -1), a tile ahead of the copies that need it.
+  auto lookup = [&](int k0) {
+    const int kp = k0 + lane;
+    const int page = kp <= key_hi ? my_table[kp / page_size] : 0;
+    return page > 0 ? page * page_size + kp % page_size : -1;
+  };
+  auto fetch = [&](int cells, __nv_bfloat16* dst, int* flags) {
+    if (warp == 0) flags[lane] = cells >= 0;
     for (int j = warp; j < NK; j += nwarps) {
-      const int kp = k0 + j;
-      int page = 0;
-      if (kp <= key_hi) page = my_table[kp / page_size];
-      const size_t at = (size_t)page * page_size + (kp % page_size);
-      if (lane == 0) flags[j] = page > 0;
+      const int cell = __shfl_sync(0xffffffffu, cells, j);
+      const bool on = cell >= 0;
+      const size_t at = on ? (size_t)cell : 0;
       for (int c = lane; c < chunks; c += 32) {
         __nv_bfloat16* to = dst + j * ld + c * 8;
-        if (page > 0 && c < chunks_lat) cp_async_16(to, latent_pages + at * rank + c * 8);
-        else if (page > 0 && c < chunks_lat + chunks_rot) cp_async_16(to, rope_pages + at * rot + (c - chunks_lat) * 8);
+        if (on && c < chunks_lat) cp_async_16(to, latent_pages + at * rank + c * 8);
+        else if (on && c < chunks_lat + chunks_rot) cp_async_16(to, rope_pages + at * rot + (c - chunks_lat) * 8);
         else *reinterpret_cast<uint4*>(to) = make_uint4(0u, 0u, 0u, 0u);
       }
     }
     cp_async_commit();
   };
   __nv_bfloat16* Kbuf[2] = {Ks, Ks + NK * ld};
-  if (key_lo <= key_hi) fetch(key_lo, Kbuf[0], there);
+  int next_cells;
+  {
+    const int first_cells = lookup(key_lo);
+    next_cells = lookup(key_lo + NK);
+    if (key_lo <= key_hi) fetch(first_cells, Kbuf[0], there);      // on its way while the queries are converted
+  }
+  // the pairs' queries as bfloat16 (rank and rot are multiples of 8, so a pair's row is whole float4s;
+  // the padding columns are zeros)
+  const int quads = Dp / 4;
+#pragma unroll 6
+  for (int i = threadIdx.x; i < AQ * quads; i += blockDim.x) {
+    const int pr = i / quads, d = (i - pr * quads) * 4;
+    const int r = pr / HG, hh = pr - r * HG;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r < rows && hh < heads && pr < BR * HG && d < Dk)
+      v = *reinterpret_cast<const float4*>(query + ((size_t)(row0 + r) * H + h0 + hh) * Dk + d);
+    uint2 packed;
+    packed.x = pack_bf16(v.x, v.y);
+    packed.y = pack_bf16(v.z, v.w);
+    *reinterpret_cast<uint2*>(Qs + pr * ld + d) = packed;
+  }
   int it = 0;
   for (int k0 = key_lo; k0 <= key_hi; k0 += NK, ++it) {
     const bool more = k0 + NK <= key_hi;
-    if (more) fetch(k0 + NK, Kbuf[(it + 1) & 1], there + ((it + 1) & 1) * NK);
+    if (more) fetch(next_cells, Kbuf[(it + 1) & 1], there + ((it + 1) & 1) * NK);
+    next_cells = lookup(k0 + 2 * NK);
     if (more) cp_async_wait<1>(); else cp_async_wait<0>();
     __syncthreads();
     const __nv_bfloat16* Kt = Kbuf[it & 1];
@@ -306,44 +316,44 @@ latent_attention_mma_kernel(float* __restrict__ out, float* __restrict__ partial
   }
 }
 
-// out[pair, :] = sum_p exp2(m_p - m) O_p / sum_p exp2(m_p - m) l_p, partitions in order.  The
-// partitions' maxima and sums are fetched side by side first; a partition that saw nothing is skipped.
+// out[pair, :] = sum_p exp2(m_p - m) O_p / sum_p exp2(m_p - m) l_p, partitions in order.  The partitions' maxima and
+// sums are fetched side by side first, every warp reduces them for itself; then a thread adds up two columns at a time,
+// eight partitions' loads under way together.  A partition that saw nothing is skipped (its O was never written).
 constexpr int MERGE_PARTS = 1024;
-__global__ void latent_merge_kernel(float* __restrict__ out, const float* __restrict__ partial, int rank, int parts) {
-  __shared__ float weight[MERGE_PARTS];
-  __shared__ float total[2];
+__global__ void __launch_bounds__(256) latent_merge_kernel(float* __restrict__ out, const float* __restrict__ partial, int rank, int parts) {
+  __shared__ float2 ml[MERGE_PARTS];
   pdl_trigger();
   pdl_wait();
-  const float* src = partial + (size_t)blockIdx.x * parts * (rank + 2);
-  for (int p = threadIdx.x; p < parts; p += blockDim.x) weight[p] = src[(size_t)p * (rank + 2)];
+  const float* src = partial + (size_t)blockIdx.x * parts * (rank + 2);      // rank is even: rows start on 8 bytes
+  for (int p = threadIdx.x; p < parts; p += blockDim.x) ml[p] = *reinterpret_cast<const float2*>(src + (size_t)p * (rank + 2));
   __syncthreads();
-  if (threadIdx.x == 0) {
-    float m = -INFINITY;
-    for (int p = 0; p < parts; ++p) m = fmaxf(m, weight[p]);
-    total[0] = m;
-  }
-  __syncthreads();
-  const float m = total[0];
-  for (int p = threadIdx.x; p < parts; p += blockDim.x) {
-    const float mp = weight[p];
-    weight[p] = mp > -INFINITY ? exp2f(mp - m) : 0.f;
-  }
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    float l = 0.f;
-    for (int p = 0; p < parts; ++p)
-      if (weight[p] > 0.f) l = fmaf(weight[p], src[(size_t)p * (rank + 2) + 1], l);
-    total[1] = l > 0.f ? 1.f / l : 0.f;
-  }
-  __syncthreads();
-  const float inv = total[1];
-  for (int d = threadIdx.x; d < rank; d += blockDim.x) {
-    float acc = 0.f;
-    for (int p = 0; p < parts; ++p) {
-      const float wp = weight[p];
-      if (wp > 0.f) acc = fmaf(wp, src[(size_t)p * (rank + 2) + 2 + d], acc);
+  const int lane = threadIdx.x & 31;
+  float m = -INFINITY, l = 0.f;
+  for (int p = lane; p < parts; p += 32) m = fmaxf(m, ml[p].x);
+  m = warp_max(m);
+  for (int p = lane; p < parts; p += 32)
+    if (ml[p].x > -INFINITY) l = fmaf(exp2f(ml[p].x - m), ml[p].y, l);
+  l = warp_sum(l);
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int d = threadIdx.x * 2; d < rank; d += blockDim.x * 2) {
+    float2 acc = make_float2(0.f, 0.f);
+    for (int p0 = 0; p0 < parts; p0 += 8) {
+      float2 v[8];
+      float w[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float mp = p0 + j < parts ? ml[p0 + j].x : -INFINITY;
+        w[j] = mp > -INFINITY ? exp2f(mp - m) : 0.f;
+        v[j] = make_float2(0.f, 0.f);
+        if (mp > -INFINITY) v[j] = *reinterpret_cast<const float2*>(src + (size_t)(p0 + j) * (rank + 2) + 2 + d);
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        acc.x = fmaf(w[j], v[j].x, acc.x);
+        acc.y = fmaf(w[j], v[j].y, acc.y);
+      }
     }
-    out[(size_t)blockIdx.x * rank + d] = acc * inv;
+    *reinterpret_cast<float2*>(out + (size_t)blockIdx.x * rank + d) = make_float2(acc.x * inv, acc.y * inv);
   }
 }
 
@@ -485,7 +495,7 @@ AYK_EXPORT int ayk_latent_attention_mma(float* out, float* partial, const float*
   if (rc != 0) return rc;
   if (launched) *launched = 1;
   if (parts > 1) {
-    ayk_launch(latent_merge_kernel, dim3(total_rows * H), dim3(rank >= 256 ? 128 : 64), 0, stream, out, (const float*)partial, rank, parts);
+    ayk_launch(latent_merge_kernel, dim3(total_rows * H), dim3(rank >= 512 ? 256 : (rank >= 256 ? 128 : 64)), 0, stream, out, (const float*)partial, rank, parts);
     if (launched) *launched = 2;
     return ayk_check_launch("ayk_latent_attention_mma (merge)");
   }

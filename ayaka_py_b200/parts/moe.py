@@ -25,7 +25,7 @@ The experts' matrices are kept stacked ([experts, 2 inner, width] with gate over
 two grouped products over the sorted rows, so nothing about the routing comes back to the host
 (``csrc/moe.cu``): on tcgen05 for bfloat16 steps of many pairs (every expert's rows padded to whole
 128-row tiles), pair by pair as matrix-vector products for a handful of pairs, on mma.sync or the
-FP32 pipes otherwise.  The shared expert's gate, up and mixing row are one dense product."""
+FP32 pipes otherwise.  The router and the shared expert's gate, up and mixing row are one dense product."""
 
 from __future__ import annotations
 
@@ -34,10 +34,6 @@ import torch
 from .. import ops
 from .base import FeedForward, TensorDecl, register_part
 from .stacked import StackedInput
-
-
-def _padded(n: int) -> int:
-    return -(-n // 8) * 8
 
 
 class MoE(FeedForward):
@@ -96,35 +92,36 @@ class MoE(FeedForward):
                 self.in_weight[e, :ff] = tensors[f"gate_{e}"]
             self.in_weight[e, -ff:] = tensors[f"up_{e}"]
             self.down_weight[e] = tensors[f"down_{e}"]
-        self.stack = StackedInput(d, [[tensors["router_weight"]]])
-        self.router_weight = self.stack.views[0]
+        groups = [[tensors["router_weight"]]]
+        if sf:
+            groups.append([tensors[name] for name in ("shared_gate", "shared_up", "shared_mix") if name in tensors])
+            self.shared_down = tensors["shared_down"]
+        self.stack = StackedInput(d, groups)
+        self._take_views()
         if "correction" in tensors:
             self.correction = tensors["correction"]
-        if sf:
-            self.shared_in = torch.zeros((_padded(2 * sf + (1 if self.shared_gated else 0)), d), dtype=first.dtype, device=first.device)
-            self.shared_in[:sf], self.shared_in[sf:2 * sf] = tensors["shared_gate"], tensors["shared_up"]
-            if self.shared_gated:
-                self.shared_in[2 * sf] = tensors["shared_mix"][0]
-            self.shared_down = tensors["shared_down"]
         for e in range(E):                         # per-expert views, as the loader's bookkeeping expects attributes
             if gated:
                 setattr(self, f"gate_{e}", self.in_weight[e, :ff])
             setattr(self, f"up_{e}", self.in_weight[e, -ff:])
             setattr(self, f"down_{e}", self.down_weight[e])
-        if sf:
-            self.shared_gate, self.shared_up = self.shared_in[:sf], self.shared_in[sf:2 * sf]
+
+    def _take_views(self) -> None:
+        self.router_weight = self.stack.views[0]
+        if self.shared_inner:
+            self.shared_gate, self.shared_up = self.stack.views[1:3]
         if self.shared_gated:
-            self.shared_mix = self.shared_in[2 * sf:2 * sf + 1]
+            self.shared_mix = self.stack.views[3]
 
     def join_input(self, weight, bias):
         """Another matrix rides in the router's product."""
         at = self.stack.join(weight, bias)
-        self.router_weight = self.stack.views[0]
+        self._take_views()
         self.joined = (at, at + weight.shape[0])
         return self.stack.views[-1]
 
     def _experts(self, h, ctx):
-        """The chosen experts' rows: (float32 rows, routing, row of every pair or None)."""
+        """The chosen experts' rows: (float32 rows, row of every pair or None, routing, the stacked product)."""
         pairs = h.shape[0] * self.top
         logits = ops.linear(h, self.stack.weight, self.stack.bias, out_dtype=torch.float32)
         if self.joined is not None:
@@ -144,19 +141,19 @@ class MoE(FeedForward):
         early = self.weigh == "input"
         if many:
             picked, rows = ops.moe_experts_tc(h, self.in_weight, self.down_weight, route, *glu, activation=act, weigh_input=early)
-            return picked, rows, route
+            return picked, rows, route, logits
         glu = glu if act is None else None
         if few:
             # a handful of pairs (a step of single tokens): every pair streams its expert's matrices on its own
             hidden = ops.moe_gemv(h, self.in_weight, route, glu=glu, activation=act, weigh_input=early)
-            return ops.moe_gemv(hidden, self.down_weight, route, glu=None), None, route                    # [T * K, d]
+            return ops.moe_gemv(hidden, self.down_weight, route, glu=None), None, route, logits            # [T * K, d]
         hidden = ops.moe_gemm(h, self.in_weight, route, glu=glu, out_dtype=self.dtype, activation=act, weigh_input=early)
-        return ops.moe_gemm(hidden, self.down_weight, route, glu=None, out_dtype=torch.float32), None, route
+        return ops.moe_gemm(hidden, self.down_weight, route, glu=None, out_dtype=torch.float32), None, route, logits
 
     def forward(self, h, residual, ctx):
         """ff(h) (+ residual), float32 [T, width].  h: rows in the compute dtype."""
-        picked, rows, route = self._experts(h, ctx)
-        shared, mix = self._shared(h)
+        picked, rows, route, product = self._experts(h, ctx)
+        shared, mix = self._shared(product)
         if shared is None:
             shared = torch.zeros((h.shape[0], self.width), dtype=torch.float32, device=h.device)
         out = ops.moe_combine(picked, route, shared, mix, rows, weighted=self.weigh == "output")
@@ -165,18 +162,19 @@ class MoE(FeedForward):
             return residual
         return out
 
-    def _shared(self, h):
-        """The shared expert's float32 rows and the column of their gates' logits; None for what there is not."""
+    def _shared(self, product):
+        """The shared expert's float32 rows and the column of their gates' logits; None for what there is not.
+        ``product``: the stacked product of the layer's rows."""
         if not self.shared_inner:
             return None, None
-        sp = ops.linear(h, self.shared_in, None, out_dtype=torch.float32)
+        sp = product[:, self.stack.starts[1]:]
         sh = ops.glu_limited(sp, self.shared_inner, self.shared_limit, self.slope, self.dtype, self.plus)
         return ops.linear(sh, self.shared_down, None, out_dtype=torch.float32), sp[:, 2 * self.shared_inner] if self.shared_gated else None
 
     def forward_rows(self, h, ctx):
         """The chosen experts' rows (and the shared expert's) themselves: their sum is left to the kernel that needs it."""
-        picked, rows, route = self._experts(h, ctx)
-        shared, mix = self._shared(h)
+        picked, rows, route, product = self._experts(h, ctx)
+        shared, mix = self._shared(product)
         return ops.PickedRows(picked, route, rows, weighted=self.weigh == "output", shared=shared, mix=mix)
 
 

@@ -44,7 +44,9 @@ the Vedadra design (talking attention and differential attention with windows, n
 every sublayer, gated feed-forward, layers that run twice) beside GPT-2, the closest model, at equal
 width, layer runs and feed-forward weights.  ``--only murutar``: the Murutar design (lightning recurrence, windowed
 rotary attention with a sink, gated residual branches, a side table per token, squared-ReLU experts) beside
-Tesozen, the closest model.
+Tesozen, the closest model.  ``--only tomodra``: the Tomodra design (latent attention in windows, layers that read
+another's latent, chunked rotary attention with learned sinks, normed sums, experts whose inputs are weighted) beside
+Tesozen in the same way.
 """
 
 from __future__ import annotations
@@ -836,7 +838,7 @@ def run_luporax(width: int, layers: int, batch: int, steps: int, warmup: int, pk
                        gbytes=min(16, 2 * rows) * 2 * width * d * 2 / 1e9, like="linear (decode)")
             picked = torch.randn(2 * rows, d, device="cuda")
             shared = torch.randn(rows, d, device="cuda")
-            sp = torch.randn(rows, ff.shared_in.shape[0], device="cuda")
+            sp = torch.randn(rows, 2 * ff.shared_inner + 8, device="cuda")
             ms = timed(lambda: ops.moe_combine(picked, route, shared, sp[:, 2 * ff.shared_inner]))
             kernel(f"weighted sum of experts ({label})", ms, gbytes=rows * d * 16 / 1e9, like="rmsnorm + residual")
             ms = timed(lambda: ops.glu_limited(sp, ff.shared_inner, 7.0, 1.702, bf))
@@ -1094,6 +1096,126 @@ def run_vedadra(width: int, layers: int, batch: int, steps: int, warmup: int, pk
     return result
 
 
+def graph_timer():
+    """fn -> median device milliseconds of one call, replayed from a CUDA graph with a flushed L2 before each replay."""
+    import torch
+
+    flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
+
+    def timed(fn, reps=9):
+        for _ in range(2):
+            fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        out = []
+        for _ in range(reps):
+            flush.fill_(1.0)
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            graph.replay()
+            b.record()
+            torch.cuda.synchronize()
+            out.append(a.elapsed_time(b))
+        return sorted(out)[len(out) // 2]
+    return timed
+
+
+def kernel_rows(pk: dict):
+    """(rows, add): ``add`` appends a kernel's time and its fraction of the measured peak that bounds it."""
+    rows = []
+
+    def add(name, model, ms, gbytes=None, gflop=None, like=None):
+        row = {"kernel": name, "model": model, "us": round(ms * 1e3, 1)}
+        if gbytes is not None:
+            row.update(gb_s=round(gbytes / (ms / 1e3), 1), frac=round(gbytes / (ms / 1e3) / pk["hbm_gbs"], 4), bound="hbm")
+        if gflop is not None:
+            row.update(tflops=round(gflop / ms, 2), frac=round(gflop / ms / pk["bf16_tflops"], 4), bound="bf16")
+        if like:
+            row["like"] = like
+        rows.append(row)
+    return rows, add
+
+
+def design_engine(config, batch: int):
+    """(model with random weights, engine) of a design's bench: room for two 1,024-token prompts and ``batch`` decoders."""
+    from ayaka_py_b200 import EngineConfig
+    from ayaka_py_b200.engine.engine import Engine
+    from ayaka_py_b200.engine.loading import random_model
+
+    model = random_model(config, 1, "bfloat16", "cuda", generate_on_device=True)
+    engine = Engine(model, EngineConfig(dtype="bfloat16", kv_pages=batch * 64 + 130, page_size=16, max_requests=max(batch, 2),
+                                        batch_tokens=2048, prefill_chunk=2048, max_model_len=1024, decode_graph=True),
+                    eos_token_id=None)
+    return model, engine
+
+
+def design_steps(model, engine, vocab: int, batch: int, steps: int, warmup: int, rs) -> dict:
+    """A prefill step of 2 x 1,024 tokens and decode steps of ``batch`` requests after ``PROMPT_LEN``-token prompts."""
+    import torch
+
+    from ayaka_py_b200 import Request, SamplingParams, StopCriteria
+    from ayaka_py_b200.engine.step import StepEntry
+
+    cache, runner = engine.cache, engine.runner
+
+    def prefill_step():
+        slots = [cache.open(f"p{i}") for i in range(2)]
+        entries = [StepEntry(sl, 0, rs.randint(0, vocab, 1024).tolist(), [1023]) for sl in slots]
+        res = cache.reserve([(e.slot, 0, 1024) for e in entries])
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        runner.run(entries)
+        b.record()
+        torch.cuda.synchronize()
+        cache.commit(res)
+        for sl in slots:
+            cache.close(sl)
+        return a.elapsed_time(b)
+    times = [prefill_step() for _ in range(7)][2:]
+    prefill_ms = sorted(times)[2]
+
+    total_new = 2 * warmup + steps + 8
+    for i in range(batch):
+        engine.submit(Request(f"d{i}", rs.randint(0, vocab, PROMPT_LEN).tolist(), SamplingParams(temperature=0.0),
+                              StopCriteria(max_tokens=total_new, ignore_eos=True)))
+    while any(st.computed < st.prompt_len for st in engine.scheduler.states.values()):
+        engine.step()
+    for _ in range(warmup):
+        engine.step()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    t0 = time.perf_counter()
+    a.record()
+    for _ in range(steps):
+        engine.step()
+    b.record()
+    torch.cuda.synchronize()
+    wall = time.perf_counter() - t0
+    decode_ms = a.elapsed_time(b) / steps
+    for rid in list(engine.scheduler.states):
+        engine.abort(rid)
+    engine.finished.clear()
+    return {"prefill_tok_s": round(2048 / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
+            "decode_tok_s": round(batch / (decode_ms / 1e3), 1), "decode_ms_per_step": round(decode_ms, 4),
+            "decode_e2e_tok_s": round(batch * steps / wall, 1), "weight_gb": round(model.weight_bytes() / 1e9, 3),
+            "kv_bytes_per_token": cache.bytes_per_token()}
+
+
+def open_kernel_step(cache, runner, lengths, starts=None):
+    """(context, reservation, slots) of a step in which request i brings lengths[i] tokens after starts[i]."""
+    from ayaka_py_b200.engine.step import StepEntry
+
+    slots = [cache.open(f"k{i}") for i in range(len(lengths))]
+    if starts:
+        cache.commit(cache.reserve([(sl, 0, st) for sl, st in zip(slots, starts)]))
+    res = cache.reserve([(sl, int(cache.length[sl]), n) for sl, n in zip(slots, lengths)])
+    ctx = runner.prepare([StepEntry(sl, int(cache.length[sl]), [0] * n, []) for sl, n in zip(slots, lengths)])
+    return ctx, res, slots
+
+
 def tesozen_document(width: int, layers: int, vocab: int = 32000) -> dict:
     """A Tesozen model of real-layer sizes: heads of 128 (four query heads to a key/value head, chunks of 512),
     an mLSTM with a 128 x 128 memory per head, a latent of 512, 16 experts in 4 groups of which 2 experts of 2
@@ -1120,98 +1242,22 @@ def run_tesozen(width: int, layers: int, batch: int, steps: int, warmup: int, pk
     import numpy as np
     import torch
 
-    from ayaka_py_b200 import EngineConfig, Request, SamplingParams, StopCriteria, ops
+    from ayaka_py_b200 import ops
     from ayaka_py_b200.config.model import LuporaxConfig, TesozenConfig
-    from ayaka_py_b200.engine.engine import Engine
-    from ayaka_py_b200.engine.loading import random_model
-    from ayaka_py_b200.engine.step import StepEntry
 
     vocab, heads = 32000, width // 128
     configs = {"tesozen": TesozenConfig.from_dict(tesozen_document(width, layers, vocab)),
                "luporax": LuporaxConfig.from_dict(luporax_document(width, layers, vocab))}
-    flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
     rs = np.random.RandomState(3)
-
-    def timed(fn, reps=9):
-        for _ in range(2):
-            fn()
-        torch.cuda.synchronize()
-        graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph):
-            fn()
-        out = []
-        for _ in range(reps):
-            flush.fill_(1.0)
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            a.record()
-            graph.replay()
-            b.record()
-            torch.cuda.synchronize()
-            out.append(a.elapsed_time(b))
-        return sorted(out)[len(out) // 2]
+    timed = graph_timer()
 
     result = {"width": width, "layers": layers, "batch": batch}
-    kernels = []
-
-    def kernel(name, model, ms, gbytes=None, gflop=None, like=None):
-        row = {"kernel": name, "model": model, "us": round(ms * 1e3, 1)}
-        if gbytes is not None:
-            row.update(gb_s=round(gbytes / (ms / 1e3), 1), frac=round(gbytes / (ms / 1e3) / pk["hbm_gbs"], 4), bound="hbm")
-        if gflop is not None:
-            row.update(tflops=round(gflop / ms, 2), frac=round(gflop / ms / pk["bf16_tflops"], 4), bound="bf16")
-        if like:
-            row["like"] = like
-        kernels.append(row)
+    kernels, kernel = kernel_rows(pk)
 
     for name, config in configs.items():
-        model = random_model(config, 1, "bfloat16", "cuda", generate_on_device=True)
-        engine = Engine(model, EngineConfig(dtype="bfloat16", kv_pages=batch * 64 + 130, page_size=16, max_requests=max(batch, 2),
-                                            batch_tokens=2048, prefill_chunk=2048, max_model_len=1024, decode_graph=True),
-                        eos_token_id=None)
+        model, engine = design_engine(config, batch)
         cache, runner = engine.cache, engine.runner
-
-        def prefill_step():
-            slots = [cache.open(f"p{i}") for i in range(2)]
-            entries = [StepEntry(sl, 0, rs.randint(0, vocab, 1024).tolist(), [1023]) for sl in slots]
-            res = cache.reserve([(e.slot, 0, 1024) for e in entries])
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            torch.cuda.synchronize()
-            a.record()
-            runner.run(entries)
-            b.record()
-            torch.cuda.synchronize()
-            cache.commit(res)
-            for sl in slots:
-                cache.close(sl)
-            return a.elapsed_time(b)
-        times = [prefill_step() for _ in range(5)][2:]
-        prefill_ms = sorted(times)[1]
-
-        total_new = 2 * warmup + steps + 8
-        for i in range(batch):
-            engine.submit(Request(f"d{i}", rs.randint(0, vocab, PROMPT_LEN).tolist(), SamplingParams(temperature=0.0),
-                                  StopCriteria(max_tokens=total_new, ignore_eos=True)))
-        while any(st.computed < st.prompt_len for st in engine.scheduler.states.values()):
-            engine.step()
-        for _ in range(warmup):
-            engine.step()
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        a.record()
-        for _ in range(steps):
-            engine.step()
-        b.record()
-        torch.cuda.synchronize()
-        wall = time.perf_counter() - t0
-        decode_ms = a.elapsed_time(b) / steps
-        result[name] = {"prefill_tok_s": round(2048 / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
-                        "decode_tok_s": round(batch / (decode_ms / 1e3), 1), "decode_ms_per_step": round(decode_ms, 4),
-                        "decode_e2e_tok_s": round(batch * steps / wall, 1), "weight_gb": round(model.weight_bytes() / 1e9, 3),
-                        "kv_bytes_per_token": cache.bytes_per_token()}
-        for rid in list(engine.scheduler.states):
-            engine.abort(rid)
-        engine.finished.clear()
+        result[name] = design_steps(model, engine, vocab, batch, steps, warmup, rs)
 
         # ---- the kernels alone, on the shapes of the two steps above
         d, T = width, 2048
@@ -1221,17 +1267,8 @@ def run_tesozen(width: int, layers: int, batch: int, steps: int, warmup: int, pk
         chunk_pairs = 2 * 2 * (512 * 513 // 2)              # two prompts of two chunks of 512
         ctx_len = PROMPT_LEN + 64
 
-        def open_step(lengths, starts=None):
-            slots = [cache.open(f"k{i}") for i in range(len(lengths))]
-            if starts:
-                res = cache.reserve([(sl, 0, st) for sl, st in zip(slots, starts)])
-                cache.commit(res)
-            res = cache.reserve([(sl, int(cache.length[sl]), n) for sl, n in zip(slots, lengths)])
-            ctx = runner.prepare([StepEntry(sl, int(cache.length[sl]), [0] * n, []) for sl, n in zip(slots, lengths)])
-            return ctx, res, slots
-
         for label, lengths, starts in (("prefill", [1024, 1024], None), ("decode", [1] * batch, [ctx_len] * batch)):
-            ctx, res, slots = open_step(lengths, starts)
+            ctx, res, slots = open_kernel_step(cache, runner, lengths, starts)
             rows = ctx.num_rows
             xr = x[:rows].contiguous()
             y = torch.randn(rows, d, device="cuda")
@@ -1400,98 +1437,22 @@ def run_murutar(width: int, layers: int, batch: int, steps: int, warmup: int, pk
     import numpy as np
     import torch
 
-    from ayaka_py_b200 import EngineConfig, Request, SamplingParams, StopCriteria, ops
+    from ayaka_py_b200 import ops
     from ayaka_py_b200.config.model import MurutarConfig, TesozenConfig
-    from ayaka_py_b200.engine.engine import Engine
-    from ayaka_py_b200.engine.loading import random_model
-    from ayaka_py_b200.engine.step import StepEntry
 
     vocab, heads = 32000, width // 128
     configs = {"murutar": MurutarConfig.from_dict(murutar_document(width, layers, vocab)),
                "tesozen": TesozenConfig.from_dict(tesozen_document(width, layers, vocab))}
-    flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
     rs = np.random.RandomState(3)
-
-    def timed(fn, reps=9):
-        for _ in range(2):
-            fn()
-        torch.cuda.synchronize()
-        graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph):
-            fn()
-        out = []
-        for _ in range(reps):
-            flush.fill_(1.0)
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            a.record()
-            graph.replay()
-            b.record()
-            torch.cuda.synchronize()
-            out.append(a.elapsed_time(b))
-        return sorted(out)[len(out) // 2]
+    timed = graph_timer()
 
     result = {"width": width, "layers": layers, "batch": batch}
-    kernels = []
-
-    def kernel(name, model, ms, gbytes=None, gflop=None, like=None):
-        row = {"kernel": name, "model": model, "us": round(ms * 1e3, 1)}
-        if gbytes is not None:
-            row.update(gb_s=round(gbytes / (ms / 1e3), 1), frac=round(gbytes / (ms / 1e3) / pk["hbm_gbs"], 4), bound="hbm")
-        if gflop is not None:
-            row.update(tflops=round(gflop / ms, 2), frac=round(gflop / ms / pk["bf16_tflops"], 4), bound="bf16")
-        if like:
-            row["like"] = like
-        kernels.append(row)
+    kernels, kernel = kernel_rows(pk)
 
     for name, config in configs.items():
-        model = random_model(config, 1, "bfloat16", "cuda", generate_on_device=True)
-        engine = Engine(model, EngineConfig(dtype="bfloat16", kv_pages=batch * 64 + 130, page_size=16, max_requests=max(batch, 2),
-                                            batch_tokens=2048, prefill_chunk=2048, max_model_len=1024, decode_graph=True),
-                        eos_token_id=None)
+        model, engine = design_engine(config, batch)
         cache, runner = engine.cache, engine.runner
-
-        def prefill_step():
-            slots = [cache.open(f"p{i}") for i in range(2)]
-            entries = [StepEntry(sl, 0, rs.randint(0, vocab, 1024).tolist(), [1023]) for sl in slots]
-            res = cache.reserve([(e.slot, 0, 1024) for e in entries])
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            torch.cuda.synchronize()
-            a.record()
-            runner.run(entries)
-            b.record()
-            torch.cuda.synchronize()
-            cache.commit(res)
-            for sl in slots:
-                cache.close(sl)
-            return a.elapsed_time(b)
-        times = [prefill_step() for _ in range(7)][2:]
-        prefill_ms = sorted(times)[2]
-
-        total_new = 2 * warmup + steps + 8
-        for i in range(batch):
-            engine.submit(Request(f"d{i}", rs.randint(0, vocab, PROMPT_LEN).tolist(), SamplingParams(temperature=0.0),
-                                  StopCriteria(max_tokens=total_new, ignore_eos=True)))
-        while any(st.computed < st.prompt_len for st in engine.scheduler.states.values()):
-            engine.step()
-        for _ in range(warmup):
-            engine.step()
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        a.record()
-        for _ in range(steps):
-            engine.step()
-        b.record()
-        torch.cuda.synchronize()
-        wall = time.perf_counter() - t0
-        decode_ms = a.elapsed_time(b) / steps
-        result[name] = {"prefill_tok_s": round(2048 / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
-                        "decode_tok_s": round(batch / (decode_ms / 1e3), 1), "decode_ms_per_step": round(decode_ms, 4),
-                        "decode_e2e_tok_s": round(batch * steps / wall, 1), "weight_gb": round(model.weight_bytes() / 1e9, 3),
-                        "kv_bytes_per_token": cache.bytes_per_token()}
-        for rid in list(engine.scheduler.states):
-            engine.abort(rid)
-        engine.finished.clear()
+        result[name] = design_steps(model, engine, vocab, batch, steps, warmup, rs)
 
         # ---- the kernels alone, on the shapes of the two steps above
         d, T = width, 2048
@@ -1499,17 +1460,8 @@ def run_murutar(width: int, layers: int, batch: int, steps: int, warmup: int, pk
         x = torch.randn(T, d, device="cuda")
         ctx_len = PROMPT_LEN + 64
 
-        def open_step(lengths, starts=None):
-            slots = [cache.open(f"k{i}") for i in range(len(lengths))]
-            if starts:
-                res = cache.reserve([(sl, 0, st) for sl, st in zip(slots, starts)])
-                cache.commit(res)
-            res = cache.reserve([(sl, int(cache.length[sl]), n) for sl, n in zip(slots, lengths)])
-            ctx = runner.prepare([StepEntry(sl, int(cache.length[sl]), [0] * n, []) for sl, n in zip(slots, lengths)])
-            return ctx, res, slots
-
         for label, lengths, starts in (("prefill", [1024, 1024], None), ("decode", [1] * batch, [ctx_len] * batch)):
-            ctx, res, slots = open_step(lengths, starts)
+            ctx, res, slots = open_kernel_step(cache, runner, lengths, starts)
             rows = ctx.num_rows
             xr = x[:rows].contiguous()
             h = xr.to(bf)
@@ -1654,6 +1606,187 @@ def run_murutar(width: int, layers: int, batch: int, steps: int, warmup: int, pk
     return result
 
 
+def tomodra_document(width: int, layers: int, vocab: int = 32000) -> dict:
+    """A Tomodra model of real-layer sizes: heads of 128 (four query heads to a key/value head, chunks of 512, half of a
+    head's dimensions turning with stretched frequencies), a latent of 512 with a rotated part of 64 in windows of 512,
+    every second latent layer reading the latent of the one before, and Tesozen's expert sizes (16 experts, 2 chosen)."""
+    heads = width // 128
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": width}, "shared": {"ff": width * 3 // 4}}
+    att = {"type": "attention", "mlp": moe,
+           "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 512},
+                     "rot": {"base": 50000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 256, "fast": 32.0, "slow": 1.0}}}}
+    lat = {"type": "latent_attention", "mlp": moe,
+           "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "mask": {"size": 512},
+                     "rot": {"base": 500000.0, "dims": 64}}}
+
+    def at(i):
+        return (att, lat, dict(lat, mixer=dict(lat["mixer"], kv_from=i - 1)), att)[i % 4]
+    return {"architecture": "Tomodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": (2.0 * layers) ** 0.25,
+            "layers": [at(i) for i in range(layers)]}
+
+
+def run_tomodra(width: int, layers: int, batch: int, steps: int, warmup: int, pk: dict) -> dict:
+    """Tomodra beside Tesozen, the closest model (latent attention, softmax attention inside chunks, experts routed by
+    sigmoid scores beside a shared one), at equal width, depth and expert sizes (bfloat16, random weights): prefill of
+    2 x 1,024 tokens in one step, decode of ``batch`` requests after 512-token prompts through the engine (CUDA graphs),
+    and the design's kernels one by one beside the like kernels of Tesozen, timed as in ``run_rakalix``."""
+    import numpy as np
+    import torch
+
+    from ayaka_py_b200 import ops
+    from ayaka_py_b200.config.model import TesozenConfig, TomodraConfig
+
+    vocab, heads = 32000, width // 128
+    configs = {"tomodra": TomodraConfig.from_dict(tomodra_document(width, layers, vocab)),
+               "tesozen": TesozenConfig.from_dict(tesozen_document(width, layers, vocab))}
+    rs = np.random.RandomState(3)
+    timed = graph_timer()
+    result = {"width": width, "layers": layers, "batch": batch}
+    kernels, kernel = kernel_rows(pk)
+    for name, config in configs.items():
+        model, engine = design_engine(config, batch)
+        cache, runner = engine.cache, engine.runner
+        result[name] = design_steps(model, engine, vocab, batch, steps, warmup, rs)
+        mine = name == "tomodra"
+
+        # ---- the kernels alone, on the shapes of the two steps above
+        d, D, R, rank = width, 128, 64 if mine else 0, 512
+        bf, f32, inf = torch.bfloat16, torch.float32, float("inf")
+        ctx_len = PROMPT_LEN + 64
+        at, lt = (0, 1) if mine else (1, 2)
+        att, lat = model.blocks[at], model.blocks[lt]
+        am, lm, ff = att.mixer, lat.mixer, lat.ffn
+        ab, lb = model.bindings[at]["mixer"], model.bindings[lt]["mixer"]
+        kp, vp = cache.kv_layer(ab.group, ab.layer)
+        rope, latent = cache.kv_layer(lb.group, lb.layer)
+        G = am.kv_heads
+        for label, lengths, starts in (("prefill", [1024, 1024], None), ("decode", [1] * batch, [ctx_len] * batch)):
+            prefill = label == "prefill"
+            ctx, res, slots = open_kernel_step(cache, runner, lengths, starts)
+            rows = ctx.num_rows
+            x, y = torch.randn(rows, d, device="cuda"), torch.randn(rows, d, device="cuda")
+            h = x.to(bf)
+            atab, ltab = ctx.tables[ab.group], ctx.tables[lb.group]
+            like = (lambda text: text) if mine else (lambda text: None)
+
+            # the stream
+            if mine:
+                ms = timed(lambda: att.norm1.sum_normed(x, y, att.copy, ctx))
+                kernel(f"sum, norm, copy ({label})", name, ms, gbytes=rows * d * 14 / 1e9, like="layer norm + residual + next layer norm")
+            else:
+                ms = timed(lambda: att.norm1b.add_normed_then(x, y, att.norm2))
+                kernel(f"layer norm + residual + next layer norm ({label})", name, ms, gbytes=rows * d * 14 / 1e9)
+
+            # the chunked attention
+            n = (am.stack.weight if mine else am.in_weight).shape[0]
+            ms = timed(lambda: ops.linear(h, am.stack.weight if mine else am.in_weight, None, out_dtype=f32))
+            kernel(f"attention's first product {rows}x{n}x{d}, 32-bit out ({label})", name, ms, gflop=2.0 * rows * n * d / 1e9,
+                   like=like("attention's first product"))
+            aproj = torch.randn(rows, n, device="cuda")
+            chunk_pairs = 2 * 2 * (512 * 513 // 2) if prefill else 0
+            seen = batch * ((ctx_len % 512) + 1)
+            if mine:
+                rot = am.rotary
+                ms = timed(lambda: ops.rotary_prepare(aproj, kp, vp, rot.freq, rot.dims, ctx, atab, heads, True, bf, gain=rot.gain, halves=rot.halves,
+                                                      q_norm=am.q_norm, k_norm=am.k_norm, eps=1e-6))
+                kernel(f"head norms, rotation, filing ({label})", name, ms, gbytes=rows * (heads + 2 * G) * D * 6 / 1e9, like="head norms + filing")
+                q = torch.randn(rows, heads * D, device="cuda").to(bf)
+                ms = timed(lambda: ops.grouped_attention(q, kp, vp, atab, ctx, heads=heads, key_heads=G, key_dim=D, scale=am.scale, chunk=am.chunk,
+                                                         sinks=am.sinks))
+                kernel(f"attention in chunks of 512 with sinks ({label})", name, ms, like="differential attention in chunks of 512",
+                       **({"gflop": chunk_pairs * heads * 2 * 256 / 1e9} if prefill else {"gbytes": seen * G * 2 * D * 2 / 1e9}))
+            else:
+                ms = timed(lambda: ops.head_norm_prepare(aproj, kp, vp, am.q_norm, am.k_norm, ctx, atab, heads, G, D, 2, (heads + G) * 2 * D,
+                                                         1e-6, True, bf))
+                kernel(f"head norms + filing ({label})", name, ms, gbytes=rows * (2 * heads + 3 * G) * D * 6 / 1e9)
+                q = torch.randn(rows, 2 * heads * D, device="cuda").to(bf)
+                gate = aproj[:, (heads + G) * 2 * D + G * D:]
+                ms = timed(lambda: ops.grouped_attention(q, kp, vp, atab, ctx, heads=2 * heads, key_heads=2 * G, key_dim=D, scale=am.scale,
+                                                         maps=2, lam=am.lam, post_scale=0.4, eps=1e-6, chunk=am.chunk, gate=gate))
+                kernel(f"differential attention in chunks of 512 ({label})", name, ms,
+                       **({"gflop": chunk_pairs * 2 * heads * 2 * 256 / 1e9} if prefill else {"gbytes": seen * G * 3 * D * 2 / 1e9}))
+
+            # the latent attention
+            n = lm.in_weight.shape[0]
+            ms = timed(lambda: ops.linear(h, lm.in_weight, None, out_dtype=f32))
+            kernel(f"latent attention's first product {rows}x{n}x{d}, 32-bit out ({label})", name, ms, gflop=2.0 * rows * n * d / 1e9,
+                   like=like("latent attention's first product"))
+            lproj = torch.randn(rows, n, device="cuda")
+            rot = lm.rotary
+            freq = rot.freq if mine else torch.zeros(1, device="cuda")
+            ms = timed(lambda: ops.latent_prepare(lproj, latent, rope, lm.down_norm, freq, 1.0, R, ctx, ltab, heads, D, R, rank, 1e-6, True,
+                                                  mine and rot.halves))
+            kernel(f"latent norm{', rotation,' if mine else ' +'} filing ({label})", name, ms,
+                   gbytes=rows * ((rank + R) * 6 + heads * R * 8) / 1e9, like=like("latent norm + filing"))
+            if mine:
+                ms = timed(lambda: ops.latent_prepare(lproj, latent, rope, None, freq, 1.0, R, ctx, ltab, heads, D, R, rank, 1e-6, False, rot.halves))
+                kernel(f"rotation of a layer that reads another's latent ({label})", name, ms, gbytes=rows * heads * R * 8 / 1e9,
+                       like="latent norm + filing")
+            query = torch.randn(rows, heads, rank + R, device="cuda")
+            plain_part = lproj[:, :heads * (D + R)].view(rows, heads, D + R)[:, :, :D]
+            ms = timed(lambda: ops.head_matmul(plain_part, lm.uk_heads, query[:, :, :rank]))
+            kernel(f"per-head product K128 N512 ({label})", name, ms, gflop=2.0 * rows * heads * D * rank / 1e9, like=like("per-head product K128 N512"))
+            ms = timed(lambda: ops.latent_attention(query, latent, rope, ltab, ctx, lm.scale, window=lm.window))
+            if prefill:
+                pairs = 2 * (sum(min(i + 1, 512) for i in range(1024)) if mine else 1024 * 1025 // 2)
+                kernel(f"latent attention{' in windows of 512' if mine else ''} (prefill)", name, ms, gflop=pairs * heads * 2 * (2 * rank + R) / 1e9,
+                       like=like("latent attention"))
+            else:
+                keys = min(512, ctx_len + 1) if mine else ctx_len + 1
+                kernel(f"latent attention{' in windows of 512' if mine else ''} + merge (decode)", name, ms, gbytes=batch * keys * (rank + R) * 2 / 1e9,
+                       like=like("latent attention"))
+            mixed = torch.randn(rows, heads, rank, device="cuda")
+            o = torch.empty(rows, heads, D, dtype=bf, device="cuda")
+            gate = None if mine else lproj[:, lm.q_width + lm.down_width:lm.q_width + lm.down_width + lm.gate_width]
+            ms = timed(lambda: ops.head_matmul(mixed, lm.uv_heads, o, gate=gate))
+            kernel(f"per-head product K512 N128{'' if mine else ' + gate'} ({label})", name, ms, gflop=2.0 * rows * heads * D * rank / 1e9,
+                   like=like("per-head product K512 N128 + gate"))
+
+            # the experts
+            n = ff.stack.weight.shape[0]
+            ms = timed(lambda: ops.linear(h, ff.stack.weight, None, out_dtype=f32))
+            kernel(f"router and shared expert's first product {rows}x{n}x{d} ({label})", name, ms, gflop=2.0 * rows * n * d / 1e9,
+                   like=like("router and shared expert's first product"))
+            logits = torch.randn(rows, 16, device="cuda")
+            scored = {"normalize": False} if mine else {"correction": ff.correction, "groups": 4, "keep": 2, "factor": 2.5}
+            ms = timed(lambda: ops.moe_route(logits, 16, 2, scored, plan=False))
+            kernel(f"routing by sigmoid scores ({label})", name, ms, gbytes=rows * (16 + 4) * 4 / 1e9, like=like("routing by sigmoid scores"))
+            route = ops.moe_route(logits, 16, 2, scored)
+            if prefill:
+                ms = timed(lambda: ops.moe_experts_tc(h, ff.in_weight, ff.down_weight, route, inf, 1.0, 0.0, weigh_input=mine))
+                kernel("experts on tcgen05: plan, gather, gate | up, silu gating, down (prefill)", name, ms, gflop=2.0 * 2 * rows * 3 * width * d / 1e9,
+                       like=like("experts on tcgen05"))
+                picked, where = ops.moe_experts_tc(h, ff.in_weight, ff.down_weight, route, inf, 1.0, 0.0)
+            else:
+                ms = timed(lambda: ops.moe_gemv(h, ff.in_weight, route, glu=(inf, 1.0, 0.0), weigh_input=mine))
+                kernel("experts' gate | up product + silu gating, pair by pair (decode)", name, ms, gbytes=2 * rows * 2 * width * d * 2 / 1e9,
+                       like=like("experts' gate | up product"))
+                hidden = ops.moe_gemv(h, ff.in_weight, route, glu=(inf, 1.0, 0.0))
+                ms = timed(lambda: ops.moe_gemv(hidden, ff.down_weight, route, glu=None))
+                kernel("experts' down product, pair by pair (decode)", name, ms, gbytes=2 * rows * width * d * 2 / 1e9, like=like("experts' down product"))
+                picked, where = ops.moe_gemv(hidden, ff.down_weight, route, glu=None), None
+            shared = torch.randn(rows, d, device="cuda")
+            if mine:
+                both = ops.PickedRows(picked, route, where, weighted=False, shared=shared, mix=torch.randn(rows, 8, device="cuda")[:, 0])
+                ms = timed(lambda: lat.norm2.sum_normed(x, both, lat.copy, ctx))
+                kernel(f"experts' sum, sum with the stream, norm, copy ({label})", name, ms, gbytes=rows * d * 22 / 1e9,
+                       like="experts' weighted sum, layer norm + residual + next layer norm")
+            else:
+                def combine():
+                    out = ops.moe_combine(picked, route, shared, None, where)
+                    return lat.norm2b.add_normed_then(x, out, lat.norm1)
+                ms = timed(combine)
+                kernel(f"experts' weighted sum, layer norm + residual + next layer norm ({label})", name, ms, gbytes=rows * d * 30 / 1e9)
+            cache.rollback(res)
+            for sl in slots:
+                cache.close(sl)
+        del engine, model
+        torch.cuda.empty_cache()
+    result["kernels"] = kernels
+    result["peaks"] = {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk["source"]}
+    return result
+
+
 def reference_line(args) -> dict:
     """The reference arm: same shape, batch, prompt length and step counts, the reference's own engine."""
     sys.path.insert(0, os.path.join(ROOT, "baseline"))
@@ -1703,8 +1836,8 @@ def main() -> int:
     parser.add_argument("--impl", default="ours", choices=("ours", "reference"))
     parser.add_argument("--no-graph", action="store_true", help="run decode steps eagerly")
     parser.add_argument("--no-points", action="store_true", help="only the decode steps at --batch")
-    parser.add_argument("--widths", default="1024,2048", help="with --only rakalix, luporax, vedadra, tesozen or murutar: the model widths to measure")
-    parser.add_argument("--only", default=None, choices=("prefill", "small", "large", "products", "rakalix", "luporax", "vedadra", "tesozen", "murutar"),
+    parser.add_argument("--widths", default="1024,2048", help="with --only rakalix, luporax, vedadra, tesozen, murutar or tomodra: the model widths to measure")
+    parser.add_argument("--only", default=None, choices=("prefill", "small", "large", "products", "rakalix", "luporax", "vedadra", "tesozen", "murutar", "tomodra"),
                         help="run one workload alone and print its numbers (for profiling): the 2,048-token prefill "
                              "step, the small shape's continuous batching, the large shape's mixed steps, or the four "
                              "products of an XL layer over row counts beside the library's matmul")
@@ -1751,6 +1884,11 @@ def main() -> int:
         for width in (int(w) for w in args.widths.split(",")):
             layers = args.layers if args.layers != XL["n_layer"] else 4
             print(json.dumps({"murutar_beside_tesozen": run_murutar(width, layers, args.batch, args.steps, args.warmup, pk)}), flush=True)
+        return 0
+    if args.only == "tomodra":
+        for width in (int(w) for w in args.widths.split(",")):
+            layers = args.layers if args.layers != XL["n_layer"] else 4
+            print(json.dumps({"tomodra_beside_tesozen": run_tomodra(width, layers, args.batch, args.steps, args.warmup, pk)}), flush=True)
         return 0
     if args.only == "products":
         for row in run_products():
