@@ -12,7 +12,7 @@
 // angles, scores, weights and sums are 32-bit.
 #include <math.h>
 
-#include "common.cuh"
+#include "vec.cuh"
 
 namespace {
 
@@ -58,14 +58,17 @@ __global__ void rotary_kernel(T* __restrict__ x, long long x_stride, const int* 
 //   q_r     = turn(q[h, dim:]) for every head     -> query[t, h, rank:]  (float32)
 // Pairs are neighbours, or with ``halves`` dimension i and i + rot_dims/2.  The row's cos and sin wait in shared memory.
 // The unrotated query parts are projected into query[t, h, :rank] by the per-head product.
-template <typename C>
+// One block per row, or with few rows several that share the row's heads (grid y; the first one also files).  VEC 4: all
+// sizes, half of the rotated dimensions (neighbours: all of them) and the rows' stride are multiples of 4, all tensors
+// 16-byte aligned.
+template <typename C, int VEC>
 __global__ void __launch_bounds__(128)
 latent_prepare_kernel(C* __restrict__ latent_pages, C* __restrict__ rope_pages, float* __restrict__ query,
                       const float* __restrict__ proj, int proj_stride, const float* __restrict__ norm_w,
                       const float* __restrict__ freq, float gain, int rot_dims, int halves, const int* __restrict__ row_req,
                       const int* __restrict__ positions, const int* __restrict__ table, int table_stride, int page_size,
                       int H, int dim, int rot, int rank, float eps, int writes) {
-  extern __shared__ float turn[];            // cos [rot_dims / 2], sin [rot_dims / 2]
+  extern __shared__ __align__(16) float turn[];            // cos [rot_dims / 2], sin [rot_dims / 2]
   __shared__ float red[4];
   pdl_trigger();
   const int t = blockIdx.x;
@@ -83,30 +86,62 @@ latent_prepare_kernel(C* __restrict__ latent_pages, C* __restrict__ rope_pages, 
   const float* row = proj + (size_t)t * proj_stride;
   const float* down = row + (size_t)H * (dim + rot);
   const int Dk = rank + rot;
-  // number e of a rotated part: u cos - v sin for the first of a pair (u, v), v cos + u sin for the second
-  auto turned = [&](const float* src, int e) {
-    if (e >= rot_dims) return src[e];
-    const int pair = halves ? (e < half ? e : e - half) : e >> 1;
-    const bool second = halves ? e >= half : (e & 1) != 0;
-    const int other = halves ? (second ? e - half : e + half) : e ^ 1;
-    const float s = turn[half + pair];
-    return fmaf(src[other], second ? s : -s, src[e] * turn[pair]);
+  // numbers e .. e + VEC - 1 of a rotated part: u cos - v sin for the first of a pair (u, v), v cos + u sin for the second
+  auto turned = [&](const float* src, int e, float (&v)[VEC]) {
+    load_n(src + e, v);
+    if (e >= rot_dims) return;
+    if (halves) {
+      const bool second = e >= half;
+      const int i0 = second ? e - half : e;
+      float o[VEC];
+      load_n(src + (second ? i0 : e + half), o);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = fmaf(o[i], second ? turn[half + i0 + i] : -turn[half + i0 + i], v[i] * turn[i0 + i]);
+    } else if (VEC == 1) {
+      const float s = turn[half + (e >> 1)];
+      v[0] = fmaf(src[e ^ 1], (e & 1) ? s : -s, v[0] * turn[e >> 1]);
+    } else {
+#pragma unroll
+      for (int i = 0; i + 1 < VEC; i += 2) {
+        const float c = turn[(e + i) >> 1], s = turn[half + ((e + i) >> 1)], a = v[i], b = v[i + 1];
+        v[i] = fmaf(b, -s, a * c);
+        v[i + 1] = fmaf(a, s, b * c);
+      }
+    }
   };
-  // rotated query parts
-  for (int i = threadIdx.x; i < H * rot; i += blockDim.x) {
-    const int h = i / rot, e = i - h * rot;
-    query[((size_t)t * H + h) * Dk + rank + e] = turned(row + (size_t)h * (dim + rot) + dim, e);
+  const int pieces = rot / VEC;              // of a head's rotated part
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * pieces; i += gridDim.y * blockDim.x) {
+    const int h = i / pieces, e = (i - h * pieces) * VEC;
+    float v[VEC];
+    turned(row + (size_t)h * (dim + rot) + dim, e, v);
+    store_n(query + ((size_t)t * H + h) * Dk + rank + e, v);
   }
-  if (!writes || page <= 0) return;      // a run step that reads another's cache; a padding lane
+  if (!writes || page <= 0 || blockIdx.y != 0) return;      // a run step that reads another's cache; a padding lane; not the first block
   const size_t at = (size_t)page * page_size + (p % page_size);
-  for (int e = threadIdx.x; e < rot; e += blockDim.x) rope_pages[at * rot + e] = from_float<C>(turned(down + rank, e));
+  for (int e = threadIdx.x * VEC; e < rot; e += blockDim.x * VEC) {
+    float v[VEC];
+    turned(down + rank, e, v);
+    store_n(rope_pages + at * rot + e, v);
+  }
   float s = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) s = fmaf(down[i], down[i], s);
+  for (int i = threadIdx.x * VEC; i < rank; i += blockDim.x * VEC) {
+    float v[VEC];
+    load_n(down + i, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) s = fmaf(v[e], v[e], s);
+  }
   s = warp_sum(s);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = s;
   __syncthreads();
   const float inv = 1.0f / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)rank + eps);
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) latent_pages[at * rank + i] = from_float<C>(down[i] * inv * norm_w[i]);
+  for (int i = threadIdx.x * VEC; i < rank; i += blockDim.x * VEC) {
+    float v[VEC], w[VEC];
+    load_n(down + i, v);
+    load_n(norm_w + i, w);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * inv * w[e];
+    store_n(latent_pages + at * rank + i, v);
+  }
 }
 
 // ------------------------------------------------------- per-head products --
@@ -424,16 +459,18 @@ AYK_EXPORT int ayk_latent_prepare(void* latent_pages, void* rope_pages, float* q
   AYK_REQUIRE(rot_dims % 2 == 0 && rot_dims <= rot, "ayk_latent_prepare: %d rotated dimensions of %d", rot_dims, rot);
   AYK_REQUIRE(rot_dims <= 8192, "ayk_latent_prepare: %d rotated dimensions", rot_dims);
   const size_t smem = (size_t)rot_dims * sizeof(float);
-  if (cache_dtype == AYK_DTYPE_F32)
-    ayk_launch(latent_prepare_kernel<float>, dim3(T), dim3(128), smem, stream, (float*)latent_pages, (float*)rope_pages, query,
-               proj, proj_stride, norm_w, freq, gain, rot_dims, halves, row_req, positions, table, table_stride, page_size, H, dim,
-               rot, rank, eps, writes);
-  else if (cache_dtype == AYK_DTYPE_BF16)
-    ayk_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(T), dim3(128), smem, stream, (__nv_bfloat16*)latent_pages,
-               (__nv_bfloat16*)rope_pages, query, proj, proj_stride, norm_w, freq, gain, rot_dims, halves, row_req, positions, table,
-               table_stride, page_size, H, dim, rot, rank, eps, writes);
-  else
-    return ayk_fail("ayk_latent_prepare: unknown dtype %d", cache_dtype);
+  const bool vec = dim % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 && rot_dims % (halves ? 8 : 4) == 0 && proj_stride % 4 == 0 &&
+                   (((uintptr_t)latent_pages | (uintptr_t)rope_pages | (uintptr_t)query | (uintptr_t)proj | (uintptr_t)norm_w) & 15) == 0;
+  const int work = (H * (rot / (vec ? 4 : 1)) + 127) / 128;
+  const int shares = T >= 64 || work <= 1 ? 1 : (work < 16 ? work : 16);
+#define AYK_LP(C, V)                                                                                                         \
+  ayk_launch(latent_prepare_kernel<C, V>, dim3(T, shares), dim3(128), smem, stream, (C*)latent_pages, (C*)rope_pages, query, \
+             proj, proj_stride, norm_w, freq, gain, rot_dims, halves, row_req, positions, table, table_stride, page_size, H, dim, \
+             rot, rank, eps, writes)
+  if (cache_dtype == AYK_DTYPE_F32) { if (vec) AYK_LP(float, 4); else AYK_LP(float, 1); }
+  else if (cache_dtype == AYK_DTYPE_BF16) { if (vec) AYK_LP(__nv_bfloat16, 4); else AYK_LP(__nv_bfloat16, 1); }
+  else return ayk_fail("ayk_latent_prepare: unknown dtype %d", cache_dtype);
+#undef AYK_LP
   return ayk_check_launch("ayk_latent_prepare");
 }
 

@@ -4,28 +4,13 @@
 // frequencies from the caller, angles, cos and sin 32-bit, cos and sin times a gain), the rest pass; the values may be
 // blended with another layer's values of the same token, v <- keep v + mix first.
 //
-// One block per row: the row's cos and sin in shared memory, a warp per head.
+// One block per row, or with few rows several that share the row's heads and values (grid y): the row's cos and sin in
+// shared memory, a warp per head.
 #include <math.h>
 
-#include "common.cuh"
+#include "vec.cuh"
 
 namespace {
-
-__device__ __forceinline__ void store_n(float* dst, const float (&v)[1]) { *dst = v[0]; }
-__device__ __forceinline__ void store_n(__nv_bfloat16* dst, const float (&v)[1]) { *dst = __float2bfloat16_rn(v[0]); }
-__device__ __forceinline__ void store_n(float* dst, const float (&v)[4]) { *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]); }
-__device__ __forceinline__ void store_n(__nv_bfloat16* dst, const float (&v)[4]) {
-  __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-  uint2 packed;
-  packed.x = *reinterpret_cast<uint32_t*>(&lo);
-  packed.y = *reinterpret_cast<uint32_t*>(&hi);
-  *reinterpret_cast<uint2*>(dst) = packed;
-}
-__device__ __forceinline__ void load_n(const float* src, float (&v)[1]) { v[0] = *src; }
-__device__ __forceinline__ void load_n(const float* src, float (&v)[4]) {
-  const float4 f = *reinterpret_cast<const float4*>(src);
-  v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-}
 
 // VEC 4: head sizes, half of the rotated dimensions (NEIGHBOURS: all of them), row strides and the columns where keys,
 // values and the other layer's values start are multiples of 4, all tensors 16-byte aligned.
@@ -56,7 +41,7 @@ rotary_prepare_kernel(C* __restrict__ qout, C* __restrict__ kpages, C* __restric
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
   const bool files = writes && page > 0;
   const size_t cell = files ? (size_t)page * page_size + (p % page_size) : 0;
-  for (int n = warp; n < H + G; n += nwarp) {
+  for (int n = blockIdx.y * nwarp + warp; n < H + G; n += gridDim.y * nwarp) {
     const bool key = n >= H;
     if (key && !files) break;
     const float* src = row + (size_t)n * D;
@@ -115,7 +100,7 @@ rotary_prepare_kernel(C* __restrict__ qout, C* __restrict__ kpages, C* __restric
   const float* vsrc = row + (size_t)(H + G) * D;
   const float* other = first ? first + (size_t)t * first_stride : nullptr;
   C* vdst = vpages + cell * (size_t)v_width;
-  for (int i = threadIdx.x * VEC; i < v_width; i += blockDim.x * VEC) {
+  for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; i < v_width; i += gridDim.y * blockDim.x * VEC) {
     float v[VEC];
     load_n(vsrc + i, v);
     if (other) {
@@ -144,8 +129,9 @@ AYK_EXPORT int ayk_rotary_prepare(void* qout, void* kpages, void* vpages, const 
   AYK_REQUIRE(!qw == !kw, "ayk_rotary_prepare: query and key norms come together");
   const bool vec = D % 4 == 0 && rot % (neighbours ? 4 : 8) == 0 && stride % 4 == 0 && v_width % 4 == 0 && (!first || first_stride % 4 == 0) &&
                    (((uintptr_t)proj | (uintptr_t)qout | (uintptr_t)kpages | (uintptr_t)vpages | (uintptr_t)first | (uintptr_t)qw | (uintptr_t)kw) & 15) == 0;
+  const int shares = T >= 64 ? 1 : ((H + G + 7) / 8 < 16 ? (H + G + 7) / 8 : 16);
 #define AYK_RP(C, V)                                                                                                     \
-  ayk_launch(neighbours ? rotary_prepare_kernel<C, V, true> : rotary_prepare_kernel<C, V, false>, dim3(T), dim3(256), smem, stream, \
+  ayk_launch(neighbours ? rotary_prepare_kernel<C, V, true> : rotary_prepare_kernel<C, V, false>, dim3(T, shares), dim3(256), smem, stream, \
              (C*)qout, (C*)kpages, (C*)vpages, proj, stride, qw, kw, eps, freq, gain, rot, first, first_stride, keep, mix, row_req, \
              positions, table, table_stride, page_size, H, G, D, v_width, writes)
   if (dtype == AYK_DTYPE_F32) { if (vec) AYK_RP(float, 4); else AYK_RP(float, 1); }
