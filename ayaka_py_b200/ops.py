@@ -508,7 +508,7 @@ def head_matmul(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch
     return out
 
 
-LATENT_WINDOW_WHOLE = 32 # a window of up to this many keys is one partition
+LATENT_WINDOW_WHOLE = 32  # a window of up to this many keys is one partition
 LATENT_PARTS = 64        # at most this many partitions of the context when every request brings one row
 
 
